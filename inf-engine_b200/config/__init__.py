@@ -3,6 +3,7 @@ from .fovunex import FovunexConfig
 from .gavatar import GavatarConfig
 from .kipezen import KipezenConfig
 from .llama import ConfigError, LlamaConfig
+from .nurilorn import NurilornConfig
 from .registry import (
     ARCHITECTURES,
     Architecture,
@@ -16,6 +17,7 @@ from .registry import (
 )
 from .spec import (
     AttentionSpec,
+    ConvAttentionSpec,
     DifferentialAttentionSpec,
     LatentAttentionSpec,
     MinGRUSpec,

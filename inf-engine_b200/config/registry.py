@@ -130,3 +130,11 @@ def _gavatar(d: dict, tensor_shapes: dict | None = None):
 
 
 register_architecture("Gavatar", _gavatar, reads_shapes=True)
+
+
+def _nurilorn(d: dict):
+    from .nurilorn import NurilornConfig
+    return NurilornConfig.from_dict(d)
+
+
+register_architecture("Nurilorn", _nurilorn)

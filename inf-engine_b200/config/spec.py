@@ -30,13 +30,15 @@ class RopeScaling:
 class NormSpec:
     """A normalisation over the last axis."""
 
-    kind: str          # "rmsnorm" | "layernorm"
+    kind: str          # "rmsnorm" | "layernorm" | "grouped_rmsnorm"
     size: int
     eps: float
     weight: str        # tensor name of the gain
     bias: str | None = None   # tensor name of the additive term ("layernorm")
     unit_offset: bool = False  # "rmsnorm": the tensor is stored around zero and the multiplier is 1 + weight
     scalar: bool = False       # "rmsnorm": the tensor is ONE number (shape ()), the multiplier of every coordinate
+    groups: int = 1            # "grouped_rmsnorm": the row is split into this many equal parts, each normed by itself
+    out_scale: float = 1.0     # "grouped_rmsnorm": a constant multiplier of the normed row
 
 
 @dataclass(frozen=True)
@@ -298,6 +300,41 @@ class ShortConvSpec:
 
 
 @dataclass(frozen=True)
+class ConvAttentionSpec(MixerSpec):
+    """Causal grouped-query softmax attention over convolved projections.
+
+    q, k, v = q_proj x, k_proj x, v_proj x, each passed through a short causal convolution over time (``q_conv``,
+    ``k_conv``, ``v_conv``: one length, no bias; None: none); then ``position`` ("rotary_partial" or "none") turns the
+    first dimensions of every query and key head.  Values, per token: ``v_keep`` keeps this layer's for later layers of
+    the same step; ``v_mix`` names a tensor of one number lambda, and v <- (1 - lambda) v + lambda v_kept with the values
+    of the last layer that kept its own.  The mixed values are what is cached.  score = q . k * scale, then ``softcap`` *
+    tanh(score / ``softcap``) when that is given; ``sink`` (a constant logit) adds exp(sink) to the softmax's denominator.
+    Head h's output is multiplied by sigmoid(``head_gate`` x)_h (tensor [n_heads, hidden]; None: no gate), then
+    ``o_proj``."""
+
+    hidden: int = 0
+    n_heads: int = 0
+    n_kv_heads: int = 0
+    head_dim: int = 0
+    v_head_dim: int = 0
+    scale: float = 1.0
+    softcap: float | None = None
+    sink: float | None = None
+    window: int | None = None      # a query sees itself and the window - 1 keys before it (None: every earlier key)
+    position: PositionSpec = PositionSpec(kind="none")
+    q_proj: str = ""
+    k_proj: str = ""
+    v_proj: str = ""
+    q_conv: ShortConvSpec | None = None
+    k_conv: ShortConvSpec | None = None
+    v_conv: ShortConvSpec | None = None
+    v_keep: bool = False
+    v_mix: str | None = None
+    head_gate: str | None = None
+    o_proj: str = ""
+
+
+@dataclass(frozen=True)
 class GatedDeltaSpec(MixerSpec):
     """The gated delta rule: a recurrent mixer with a ``head_dim x v_head_dim`` float32 state per head.
 
@@ -435,7 +472,7 @@ class PolyNormMLPSpec(FeedForwardSpec):
 
 @dataclass(frozen=True)
 class RoutedExpertsSpec(FeedForwardSpec):
-    """A mixture of gated feed-forward experts with a sigmoid router.
+    """A mixture of gated feed-forward experts with a sigmoid or a softmax router.
 
     Router scores s = sigmoid(router x) in float32; an expert's choice score is s + ``correction``.  The experts
     form ``n_groups`` groups of neighbours; a group's score is the sum of its two largest choice scores, and only
@@ -459,8 +496,15 @@ class RoutedExpertsSpec(FeedForwardSpec):
     shared_gate: str | None = None
     # ``score`` "softmax_top": the logits are router x + ``router_bias`` (float32); the ``top`` largest are chosen (no
     # groups, no correction) and their weights are the softmax over the chosen logits alone, times ``route_scale``.
+    # ``score`` "softmax": everything as for "sigmoid", with the softmax of router x over all experts as the scores.
     score: str = "sigmoid"
     router_bias: str | None = None
+    group_score: str = "top2_sum"  # a group's score: the sum of its two largest choice scores, or "max": the largest
+    # the experts' activation, as ``GatedMLPSpec`` states it
+    activation: str = "silu"
+    act_alpha: float = 1.0
+    act_limit: float = 0.0
+    up_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -486,6 +530,11 @@ class BlockSpec:
     mixer_out_norm: NormSpec | None = None
     ff_out_norm: NormSpec | None = None
     token_shift: str | None = None
+    # "scaled_prenorm": x += residual_mult * scale * part(norm(x)), ``scale`` a learned number per coordinate (tensors
+    # [hidden] for the mixer and the feed-forward; None: 1)
+    residual_mult: float = 1.0
+    mixer_scale: str | None = None
+    ff_scale: str | None = None
 
 
 @dataclass(frozen=True)
@@ -516,6 +565,7 @@ class ModelSpec:
     head: str | None                         # tensor name, or None: tied to the embedding
     optional_tensors: tuple[str, ...] = field(default_factory=tuple)  # present-but-unused names tolerated
     kind: str = "decoder"                    # which registered top level puts the parts together
+    embedding_scale: float = 1.0             # multiplier of the token embedding
 
 
 @dataclass(frozen=True)
@@ -537,7 +587,6 @@ class ReinjectDecoderSpec(ModelSpec):
     right before each schedule entry that ``reinject_before`` names (a group of layers run several times in a row takes
     the embedding anew at the start of every pass but the first)."""
 
-    embedding_scale: float = 1.0
     reinject_before: tuple[int, ...] = ()
     kind: str = "reinject_decoder"
 
@@ -550,7 +599,6 @@ class PassOffsetDecoderSpec(ModelSpec):
     pairs, and row r of the tensor ``pass_offsets`` ([rows, hidden]) is added before that entry runs (a group of layers
     run several times in a row takes the vector of its pass at the start of each pass, the first too)."""
 
-    embedding_scale: float = 1.0
     sinusoid_base: float = 0.0
     pass_offsets: str | None = None
     offset_before: tuple[tuple[int, int], ...] = ()

@@ -21,7 +21,8 @@
 // p sees keys from floor(p / chunk) * chunk on only (chunks are counted from the sequence's start, whatever the cut).
 // Several key heads may share one value head (`n_v_heads` less than the key heads: two score maps over the same
 // values), and the values may be the first dimensions of the key rows themselves (`v_row`: a compressed key/value
-// vector that is stored once).
+// vector that is stored once).  A score may be capped (softcap * tanh(s / softcap)), and a head's output may pass a
+// sigmoid gate of one number a head.
 //
 // Work split: a block takes one (request, kv head) and a tile of 32
 // (token, head-in-group) pairs, so the `group` query heads that share a kv head
@@ -61,7 +62,18 @@ struct AttnGeneralParams {
                             // when the values are the first dimensions of the keys and both pools are one)
   const float* sink;        // [n_heads] or null: the softmax's denominator also holds exp(sink[head]): a learned
                             // logit beside the keys' scores that `scale` does not multiply and that weighs nothing
+  float softcap;            // > 0: a score s (scaled, before any bias) becomes softcap * tanh(s / softcap)
+  const void* gate;         // [tokens, n_heads] of the storage type or null: a head's output times sigmoid(gate)
+  int gate_stride;
 };
+
+__device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
+
+template <typename T>
+__device__ __forceinline__ float head_gate(const AttnGeneralParams& p, int token, int head) {
+  if (p.gate == nullptr) return 1.f;
+  return 1.f / (1.f + expf(-to_f32(((const T*)p.gate)[(size_t)token * p.gate_stride + head])));
+}
 
 // the normaliser of a row whose visible keys gave the sum l at the maximum m, with the sink's term added
 __device__ __forceinline__ float inv_with_sink(float l, float m, const float* sink, int head, float out_scale) {
@@ -187,7 +199,7 @@ __global__ void __launch_bounds__(AG_THREADS) attention_general_kernel(AttnGener
       const float* kr = Ks + kk * ldq;
       for (int d = 0; d < hd; ++d) dot += qr[d] * kr[d];
       const bool visible = row_valid && kp <= my_limit && kp >= my_chunk0 && (kp >= my_first || kp < keep);
-      float sc = dot * my_scale;
+      float sc = capped(dot * my_scale, p.softcap);
       if (visible && my_bias != nullptr) sc += my_bias[min(my_limit - kp, p.bias_dists - 1)];
       s[jj] = visible ? sc : -INFINITY;
       tile_max = fmaxf(tile_max, s[jj]);
@@ -231,7 +243,7 @@ __global__ void __launch_bounds__(AG_THREADS) attention_general_kernel(AttnGener
   if (row_valid) {
     const int j = my_pair - my_t * group;
     T* o = (T*)p.out + (size_t)(q0 + my_t) * p.out_stride + (c * group + j) * hdv;
-    const float inv = inv_with_sink(l_run, m_run, p.sink, my_head, p.out_scale);
+    const float inv = inv_with_sink(l_run, m_run, p.sink, my_head, p.out_scale) * head_gate<T>(p, q0 + my_t, my_head);
 #pragma unroll
     for (int i = 0; i < AG_MAX_ACC; ++i)
       if (i < n_acc && sub + 8 * i < hdv) o[sub + 8 * i] = from_f32<T>(acc[i] * inv);
@@ -245,7 +257,7 @@ extern "C" int ie_attention_general(const void* q, void* out, const void* kpool,
                                     int page_size, int window, float scale, int act_dtype, const float* score_bias,
                                     int bias_dists, const float* head_scale, int hd_v, int keep_first,
                                     float out_scale, int chunk, int n_v_heads, int v_row, const float* sink,
-                                    cudaStream_t stream) {
+                                    float softcap, const void* gate, int gate_stride, cudaStream_t stream) {
   if (n_work <= 0) return IE_OK;
   if (hd_v <= 0) hd_v = hd;
   if (hd <= 0 || hd > 8 * AG_MAX_ACC || hd_v > 8 * AG_MAX_ACC) return IE_BAD_SIZE;
@@ -256,6 +268,7 @@ extern "C" int ie_attention_general(const void* q, void* out, const void* kpool,
   if (n_kv_heads % n_v_heads || v_row < hd_v || chunk < 0 || (chunk > 0 && keep_first > 0)) return IE_BAD_SIZE;
   AttnGeneralParams p;
   p.chunk = chunk; p.n_v_heads = n_v_heads; p.v_row = v_row; p.sink = sink;
+  p.softcap = softcap; p.gate = gate; p.gate_stride = gate_stride;
   p.q = q; p.out = out; p.kpool = kpool; p.vpool = vpool; p.block_table = block_table;
   p.q_start = q_start; p.ctx_before = ctx_before; p.work_req = work_req; p.work_pair0 = work_pair0;
   p.q_stride = q_stride; p.out_stride = out_stride; p.table_stride = table_stride;
@@ -367,7 +380,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) attention_rows_kernel(AttnGener
       if (page >= 0) {
         at = ((long long)page * p.n_kv_heads + c) * p.page_size + (kp % p.page_size);
         vat_mine = ((long long)page * p.n_v_heads + cv) * p.page_size + (kp % p.page_size);
-        sc = key_dot(kpool + at * hd, qs, hd) * my_scale;
+        sc = capped(key_dot(kpool + at * hd, qs, hd) * my_scale, p.softcap);
         if (my_bias != nullptr) sc += my_bias[min(limit - kp, p.bias_dists - 1)];
       }
     }
@@ -419,7 +432,7 @@ __global__ void __launch_bounds__(AR_WARPS * 32) attention_rows_kernel(AttnGener
   float l_all = 0.f;
 #pragma unroll
   for (int w = 0; w < AR_WARPS; ++w) l_all += s_m[w] == -INFINITY ? 0.f : s_l[w] * expf(s_m[w] - m_all);
-  const float inv = inv_with_sink(l_all, m_all, p.sink, head, p.out_scale);
+  const float inv = inv_with_sink(l_all, m_all, p.sink, head, p.out_scale) * head_gate<T>(p, n, head);
   T* o = (T*)p.out + (size_t)n * p.out_stride + head * hdv;
   for (int d = threadIdx.x; d < hdv; d += AR_WARPS * 32) {
     float total = 0.f;
@@ -435,7 +448,8 @@ extern "C" int ie_attention_rows(const void* q, void* out, const void* kpool, co
                                  int n_tokens, int n_requests, int max_rows, int n_heads, int n_kv_heads, int hd,
                                  int page_size, int window, float scale, int act_dtype, const float* score_bias,
                                  int bias_dists, const float* head_scale, int hd_v, int keep_first, float out_scale,
-                                 int chunk, int n_v_heads, int v_row, const float* sink, cudaStream_t stream) {
+                                 int chunk, int n_v_heads, int v_row, const float* sink, float softcap, const void* gate,
+                                 int gate_stride, cudaStream_t stream) {
   if (n_tokens <= 0 || n_requests <= 0) return IE_OK;
   if (hd_v <= 0) hd_v = hd;
   if (hd <= 0 || hd > 32 * AR_MAX_PER_LANE || hd_v > 32 * AR_MAX_PER_LANE) return IE_BAD_SIZE;
@@ -446,6 +460,7 @@ extern "C" int ie_attention_rows(const void* q, void* out, const void* kpool, co
   if (n_kv_heads % n_v_heads || v_row < hd_v || chunk < 0 || (chunk > 0 && keep_first > 0)) return IE_BAD_SIZE;
   AttnGeneralParams p;
   p.chunk = chunk; p.n_v_heads = n_v_heads; p.v_row = v_row; p.sink = sink;
+  p.softcap = softcap; p.gate = gate; p.gate_stride = gate_stride;
   p.q = q; p.out = out; p.kpool = kpool; p.vpool = vpool; p.block_table = block_table;
   p.q_start = q_start; p.ctx_before = ctx_before; p.work_req = nullptr; p.work_pair0 = nullptr;
   p.q_stride = q_stride; p.out_stride = out_stride; p.table_stride = table_stride;

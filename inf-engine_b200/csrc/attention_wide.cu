@@ -21,6 +21,9 @@
 #ifndef IE_AW_DV
 #define IE_AW_DV 64
 #endif
+#ifndef IE_AW_CAP
+#define IE_AW_CAP 0      // 1: scores pass softcap * tanh(s / softcap) (a build of its own: the others do not pay for it)
+#endif
 
 namespace {
 
@@ -50,6 +53,9 @@ struct WideParams {
   int v_row;       // elements between two value rows of the value pool
   int alias;       // the values are the first DV dimensions of the key rows: the key tile is the value tile
   float scale_log2;
+  float cap_in, cap_out;   // the build with capped scores: 2 log2 e scale / softcap, and softcap log2 e
+  const bf16* gate;        // [tokens, n_heads] or null: a head's output times sigmoid(gate)
+  int gate_stride;
   // without a work list (work_req null): block x is tile x % tiles of request x / tiles, and only requests that bring
   // at most max_rows (token, head-in-group) pairs take part (decode tokens; the others are a work list's)
   int tiles, max_rows;
@@ -131,6 +137,21 @@ __device__ __forceinline__ float wide_inv(float l, float m, const float* sink, i
   const float m2 = fmaxf(m, sk);
   const float f = exp2f(m - m2);
   return f / (l * f + exp2f(sk - m2));
+}
+
+// softcap * tanh(s / softcap) in the exponent's base-2 units, tanh(z) = 1 - 2 / (1 + e^(2 z)): off by a few units of the
+// last place of 1 at most, times softcap, which is the size of the rounding of a score near the cap
+__device__ __forceinline__ float score_log2(float dot, const WideParams& p) {
+#if IE_AW_CAP
+  return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(dot * p.cap_in)));
+#else
+  return dot * p.scale_log2;
+#endif
+}
+
+__device__ __forceinline__ float wide_gate(const WideParams& p, int token, int head) {
+  if (p.gate == nullptr) return 1.f;
+  return 1.f / (1.f + expf(-to_f32(p.gate[(size_t)token * p.gate_stride + head])));
 }
 
 __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
@@ -243,7 +264,7 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
         const int h = e >> 1;
         const int kp = kt + nt * 8 + 2 * t4 + (e & 1);
         const bool vis = kp >= lo[h] && kp <= limit[h];
-        const float v = vis ? s[nt][e] * p.scale_log2 : -INFINITY;
+        const float v = vis ? score_log2(s[nt][e], p) : -INFINITY;
         s[nt][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -325,7 +346,7 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
     l += __shfl_xor_sync(0xffffffffu, l, 2);
     if (pr_[h] >= n_pairs) continue;
     const int t = pr_[h] / group, j = pr_[h] - t * group;
-    const float inv = wide_inv(l, m_run[h], p.sink, c * group + j);
+    const float inv = wide_inv(l, m_run[h], p.sink, c * group + j) * wide_gate(p, q0 + t, c * group + j);
     bf16* dst = p.out + (size_t)(q0 + t) * p.out_stride + (size_t)(c * group + j) * DV + 2 * t4;
 #pragma unroll
     for (int i = 0; i < NT_O; ++i)
@@ -381,7 +402,7 @@ __global__ void __launch_bounds__(THREADS) attention_wide_merge_kernel(WideParam
   }
   const int pr = pair0 + r;
   const int t = pr / group, j = pr - t * group;
-  const float inv = wide_inv(l_all, m_all, p.sink, c * group + j);
+  const float inv = wide_inv(l_all, m_all, p.sink, c * group + j) * wide_gate(p, q0 + t, c * group + j);
   bf16* dst = p.out + (size_t)(q0 + t) * p.out_stride + (size_t)(c * group + j) * DV;
 #pragma unroll
   for (int i = 0; i < MERGE_SLOTS; ++i) {
@@ -396,11 +417,13 @@ extern "C" int ie_attention_wide_key_dim() { return DK; }
 extern "C" int ie_attention_wide_value_dim() { return DV; }
 extern "C" int ie_attention_wide_rows() { return BM; }
 extern "C" int ie_attention_wide_keys() { return BN; }
+extern "C" int ie_attention_wide_capped() { return IE_AW_CAP; }
 
 static int wide_params(WideParams& p, const void* q, void* out, const void* kpool, const void* vpool, const int* block_table,
                        const int* q_start, const int* ctx_before, int q_stride, int out_stride, int table_stride, int n_heads,
                        int n_kv_heads, int page_size, int window, float scale, int chunk, int n_v_heads, int v_row,
-                       const float* sink) {
+                       const float* sink, float softcap, const void* gate, int gate_stride) {
+  if ((softcap > 0.f) != (IE_AW_CAP != 0)) return IE_BAD_SIZE;
   if (n_kv_heads <= 0 || n_heads % n_kv_heads || page_size <= 0 || window < 0 || chunk < 0) return IE_BAD_SIZE;
   if (n_v_heads <= 0) n_v_heads = n_kv_heads;
   if (v_row <= 0) v_row = DV;
@@ -416,6 +439,9 @@ static int wide_params(WideParams& p, const void* q, void* out, const void* kpoo
   p.n_v_heads = n_v_heads; p.v_row = v_row; p.sink = sink;
   p.alias = (vpool == kpool && v_row == DK && n_v_heads == n_kv_heads && DV <= DK) ? 1 : 0;
   p.scale_log2 = scale * LOG2E;
+  p.cap_in = softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f;
+  p.cap_out = softcap * LOG2E;
+  p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
   p.tiles = 1; p.max_rows = 0; p.n_splits = 1; p.split_keys = 0; p.part_o = nullptr; p.part_ml = nullptr;
   return IE_OK;
 }
@@ -428,12 +454,14 @@ extern "C" int ie_attention_wide(const void* q, void* out, const void* kpool, co
                                  const int* q_start, const int* ctx_before, const int* work_req, const int* work_pair0,
                                  int q_stride, int out_stride, int table_stride, int n_work, int n_heads, int n_kv_heads,
                                  int page_size, int window, float scale, int chunk, int n_v_heads, int v_row,
-                                 const float* sink, cudaStream_t stream) {
+                                 const float* sink, float softcap, const void* gate, int gate_stride,
+                                 cudaStream_t stream) {
   if (n_work <= 0) return IE_OK;
   if (work_req == nullptr || work_pair0 == nullptr) return IE_BAD_SIZE;
   WideParams p;
   const int rc = wide_params(p, q, out, kpool, vpool, block_table, q_start, ctx_before, q_stride, out_stride, table_stride,
-                             n_heads, n_kv_heads, page_size, window, scale, chunk, n_v_heads, v_row, sink);
+                             n_heads, n_kv_heads, page_size, window, scale, chunk, n_v_heads, v_row, sink, softcap, gate,
+                             gate_stride);
   if (rc != IE_OK) return rc;
   p.work_req = work_req; p.work_pair0 = work_pair0;
   const size_t smem = wide_smem(p);
@@ -457,13 +485,14 @@ extern "C" int ie_attention_wide_small(const void* q, void* out, const void* kpo
                                        int table_stride, int n_requests, int max_rows, int n_heads, int n_kv_heads,
                                        int page_size, int window, float scale, int chunk, int n_v_heads, int v_row,
                                        int n_splits, int split_keys, float* scratch, const float* sink,
-                                       cudaStream_t stream) {
+                                       float softcap, const void* gate, int gate_stride, cudaStream_t stream) {
   if (n_requests <= 0) return IE_OK;
   if (max_rows <= 0 || n_splits <= 0 || n_splits > 65535) return IE_BAD_SIZE;
   if (n_splits > 1 && (split_keys <= 0 || split_keys % BN || scratch == nullptr)) return IE_BAD_SIZE;
   WideParams p;
   const int rc = wide_params(p, q, out, kpool, vpool, block_table, q_start, ctx_before, q_stride, out_stride, table_stride,
-                             n_heads, n_kv_heads, page_size, window, scale, chunk, n_v_heads, v_row, sink);
+                             n_heads, n_kv_heads, page_size, window, scale, chunk, n_v_heads, v_row, sink, softcap, gate,
+                             gate_stride);
   if (rc != IE_OK) return rc;
   p.tiles = (max_rows + BM - 1) / BM; p.max_rows = max_rows; p.n_splits = n_splits; p.split_keys = split_keys;
   const size_t n_parts = (size_t)n_requests * p.tiles * n_kv_heads * n_splits;

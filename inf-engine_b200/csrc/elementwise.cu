@@ -5,11 +5,11 @@
 #include "common.cuh"
 
 // ------------------------------------------------------------------ embedding
-// residual[n, :] = table[ids[n], :]  (the reference gathers rows without
-// scaling, engine/llama_model.py:128).  The residual stream is float32.
+// residual[n, :] = table[ids[n], :] * scale  (the reference gathers rows without
+// scaling, engine/llama_model.py:128: scale 1).  The residual stream is float32.
 template <typename TW>
 __global__ void embed_gather_kernel(const int* __restrict__ ids, const TW* __restrict__ table,
-                                    float* __restrict__ residual, int d, int vocab) {
+                                    float* __restrict__ residual, int d, int vocab, float scale) {
   pdl_trigger();
   pdl_wait();
   const int n = blockIdx.x;
@@ -20,17 +20,17 @@ __global__ void embed_gather_kernel(const int* __restrict__ ids, const TW* __res
 #endif
   const TW* row = table + (size_t)(ok ? id : 0) * d;
   float* out = residual + (size_t)n * d;
-  for (int i = threadIdx.x; i < d; i += blockDim.x) out[i] = ok ? to_f32(row[i]) : 0.f;
+  for (int i = threadIdx.x; i < d; i += blockDim.x) out[i] = ok ? to_f32(row[i]) * scale : 0.f;
 }
 
 extern "C" int ie_embed_gather(const int* ids, const void* table, int table_dtype, float* residual,
-                               int n_tokens, int d, int vocab, cudaStream_t stream) {
+                               int n_tokens, int d, int vocab, float scale, cudaStream_t stream) {
   if (n_tokens <= 0) return IE_OK;
   const int threads = d >= 1024 ? 256 : 128;
   if (table_dtype == IE_F32)
-    return launch_k(embed_gather_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, residual, d, vocab);
+    return launch_k(embed_gather_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, residual, d, vocab, scale);
   if (table_dtype == IE_BF16)
-    return launch_k(embed_gather_kernel<bf16>, n_tokens, threads, 0, stream, ids, (const bf16*)table, residual, d, vocab);
+    return launch_k(embed_gather_kernel<bf16>, n_tokens, threads, 0, stream, ids, (const bf16*)table, residual, d, vocab, scale);
   return IE_BAD_DTYPE;
 }
 

@@ -1,9 +1,11 @@
 // A mixture of feed-forward experts on the device, without a trip to the host:
 //   route    per token, from float32 router logits: sigmoid scores, a correction added for the choice only, the best
 //            groups of neighbouring experts kept, the top experts among them, their normalised weights, and the
-//            shared expert's gate; or (mode 1) the largest logits, a bias added, and the softmax over those alone;
+//            shared expert's gate; or (mode 1) the largest logits, a bias added, and the softmax over those alone; or
+//            (mode 2) as mode 0 with the softmax over all experts as the scores.  A group's score is the sum of its two
+//            largest choice scores or (group_max) the largest one;
 //   sort     the (token, choice) pairs ordered by expert, and a table of row tiles, none of which spans two experts;
-//   product  C[pair] = A[token of pair] W[expert of pair]^T over those tiles, optionally with silu(gate) * up in the
+//   product  C[pair] = A[token of pair] W[expert of pair]^T over those tiles, optionally with the gated activation in the
 //            epilogue: on CUDA cores (float32 products and sums, every output one accumulator that walks k upward) for
 //            the 32-bit path, on tensor cores (mma.sync, float32 accumulators) for bfloat16 operands; either way a
 //            row's result does not depend on which tile or step it is in;
@@ -17,7 +19,7 @@ template <typename TW>
 __global__ void __launch_bounds__(128)
 route_kernel(const float* __restrict__ logits, int ld, const TW* __restrict__ correction, int* __restrict__ ids,
              float* __restrict__ weights, float* __restrict__ gate, int n_tokens, int n_experts, int top, int n_groups,
-             int keep_groups, float route_scale, float weight_eps, int gate_col, int mode) {
+             int keep_groups, float route_scale, float weight_eps, int gate_col, int mode, int group_max) {
   extern __shared__ float sm[];
   pdl_trigger();
   pdl_wait();
@@ -28,10 +30,17 @@ route_kernel(const float* __restrict__ logits, int ld, const TW* __restrict__ co
   float* choice = score + n_experts;                               // s + correction, -inf once taken or shut out
   float* gscore = choice + n_experts;
   const float* z = logits + (size_t)t * ld;
+  float z_max = -INFINITY, z_inv = 0.f;
+  if (mode == 2) {
+    for (int e = lane; e < n_experts; e += 32) z_max = fmaxf(z_max, z[e]);
+    z_max = warp_max(z_max);
+    for (int e = lane; e < n_experts; e += 32) z_inv += expf(z[e] - z_max);
+    z_inv = 1.f / warp_sum(z_inv);
+  }
   for (int e = lane; e < n_experts; e += 32) {
     const float cor = correction ? to_f32(correction[e]) : 0.f;
     // mode 1: the logits themselves (plus their bias) are both what is compared and what the weights are made of
-    const float s = mode == 1 ? z[e] + cor : 1.f / (1.f + expf(-z[e]));
+    const float s = mode == 1 ? z[e] + cor : (mode == 2 ? expf(z[e] - z_max) * z_inv : 1.f / (1.f + expf(-z[e])));
     score[e] = s;
     choice[e] = mode == 1 ? s : s + cor;
   }
@@ -44,7 +53,7 @@ route_kernel(const float* __restrict__ logits, int ld, const TW* __restrict__ co
         const float c = choice[e];
         if (c > a) { b = a; a = c; } else if (c > b) b = c;
       }
-      gscore[g] = per > 1 ? a + b : a;
+      gscore[g] = per > 1 && !group_max ? a + b : a;
     }
     __syncwarp();
     // the groups that stay: keep_groups times the largest score left; the others are shut out afterwards
@@ -113,7 +122,7 @@ route_kernel(const float* __restrict__ logits, int ld, const TW* __restrict__ co
 
 extern "C" int ie_moe_route(const float* logits, int ld, const void* correction, int w_dtype, int* ids, float* weights,
                             float* gate, int n_tokens, int n_experts, int top, int n_groups, int keep_groups,
-                            float route_scale, float weight_eps, int gate_col, int mode, cudaStream_t stream) {
+                            float route_scale, float weight_eps, int gate_col, int mode, int group_max, cudaStream_t stream) {
   if (n_tokens <= 0) return IE_OK;
   if (n_experts <= 0 || top <= 0 || top > n_experts || n_groups <= 0 || n_experts % n_groups || keep_groups <= 0 ||
       keep_groups > n_groups)
@@ -123,10 +132,10 @@ extern "C" int ie_moe_route(const float* logits, int ld, const void* correction,
   const unsigned blocks = (unsigned)((n_tokens + 3) / 4);
   if (w_dtype == IE_F32)
     return launch_k(route_kernel<float>, blocks, 128, smem, stream, logits, ld, (const float*)correction, ids, weights,
-                    gate, n_tokens, n_experts, top, n_groups, keep_groups, route_scale, weight_eps, gate_col, mode);
+                    gate, n_tokens, n_experts, top, n_groups, keep_groups, route_scale, weight_eps, gate_col, mode, group_max);
   if (w_dtype == IE_BF16)
     return launch_k(route_kernel<bf16>, blocks, 128, smem, stream, logits, ld, (const bf16*)correction, ids, weights,
-                    gate, n_tokens, n_experts, top, n_groups, keep_groups, route_scale, weight_eps, gate_col, mode);
+                    gate, n_tokens, n_experts, top, n_groups, keep_groups, route_scale, weight_eps, gate_col, mode, group_max);
   return IE_BAD_DTYPE;
 }
 
@@ -181,6 +190,17 @@ extern "C" int ie_moe_sort(const int* ids, int n_pairs, int n_experts, int tile_
 }
 
 // ------------------------------------------------------------------ grouped product
+// The activation of a gated expert: g' sigmoid(alpha g') * (u' + up_offset), g' = min(g, limit) and u' = u clamped to
+// [-limit, limit] (silu(g) * u: alpha 1, an infinite limit, no offset).
+struct GluAct {
+  float alpha, limit, up_offset;
+};
+__device__ __forceinline__ float glu(const GluAct& a, float g, float u) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit) + a.up_offset;
+  return g / (1.f + expf(-a.alpha * g)) * u;
+}
+
 #define MG_BM 64
 #define MG_BN 64
 #define MG_BK 16
@@ -189,12 +209,12 @@ extern "C" int ie_moe_sort(const int* ids, int n_pairs, int n_experts, int tile_
 // A row of tile (expert e, positions pos0 .. pos0 + rows): gather = 1: row sorted[pos] / top of A (a token's
 // activations); gather = 0: row pos of A (what the product before left in sorted order).  C row: scatter = 1: row
 // sorted[pos] (the pair's own place), else row pos.  W is [experts, N, K].  epi 1: columns alternate gate, up and the
-// output is silu(gate) * up, N / 2 wide.
+// output is the gated activation, N / 2 wide.
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(MG_THREADS)
 moe_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restrict__ C, const int* __restrict__ sorted,
                 const int* __restrict__ tiles, int N, int K, int lda, int ldc, long long w_expert_stride, int top,
-                int gather, int scatter, int epi) {
+                int gather, int scatter, int epi, GluAct act) {
   pdl_trigger();
   pdl_wait();
   __shared__ float As[MG_BK][MG_BM + 4];
@@ -258,8 +278,7 @@ moe_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restri
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
         if (n + 1 < N) {
-          const float g = acc[i][j];
-          C[(size_t)cr * ldc + (n >> 1)] = from_f32<TC>(g / (1.f + expf(-g)) * acc[i][j + 1]);
+          C[(size_t)cr * ldc + (n >> 1)] = from_f32<TC>(glu(act, acc[i][j], acc[i][j + 1]));
         }
       }
     } else {
@@ -275,10 +294,10 @@ moe_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restri
 template <typename TA, typename TW, typename TC>
 static int launch_moe_gemm(const void* A, const void* W, void* C, const int* sorted, const int* tiles, int max_tiles,
                            int N, int K, int lda, int ldc, long long wes, int top, int gather, int scatter, int epi,
-                           cudaStream_t stream) {
+                           GluAct act, cudaStream_t stream) {
   dim3 grid((N + MG_BN - 1) / MG_BN, max_tiles);
   return launch_k(moe_gemm_kernel<TA, TW, TC>, grid, MG_THREADS, 0, stream, (const TA*)A, (const TW*)W, (TC*)C, sorted,
-                  tiles, N, K, lda, ldc, wes, top, gather, scatter, epi);
+                  tiles, N, K, lda, ldc, wes, top, gather, scatter, epi, act);
 }
 
 // ---- the same product on tensor cores, for bfloat16 operands (mma.sync m16n8k16, float32 accumulators): a block
@@ -311,7 +330,7 @@ template <typename TC>
 __global__ void __launch_bounds__(MM_THREADS)
 moe_gemm_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* __restrict__ C,
                     const int* __restrict__ sorted, const int* __restrict__ tiles, int N, int K, int lda, int ldc,
-                    long long w_expert_stride, int top, int gather, int scatter, int epi) {
+                    long long w_expert_stride, int top, int gather, int scatter, int epi, GluAct act) {
   pdl_trigger();
   pdl_wait();
   __shared__ __align__(16) bf16 As[2][MM_BM * MM_LD];
@@ -394,7 +413,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* 
         const int n = n0 + wn * 32 + nt * 8 + (lane & 3) * 2;
         const float x0 = acc[mt][nt][half * 2], x1 = acc[mt][nt][half * 2 + 1];
         if (epi == 1) {
-          if (n + 1 < N) C[(size_t)cr * ldc + (n >> 1)] = from_f32<TC>(x0 / (1.f + expf(-x0)) * x1);
+          if (n + 1 < N) C[(size_t)cr * ldc + (n >> 1)] = from_f32<TC>(glu(act, x0, x1));
         } else {
           if (n < N) C[(size_t)cr * ldc + n] = from_f32<TC>(x0);
           if (n + 1 < N) C[(size_t)cr * ldc + n + 1] = from_f32<TC>(x1);
@@ -408,7 +427,9 @@ extern "C" int ie_moe_tile_rows() { return MG_BM; }
 
 extern "C" int ie_moe_gemm(const void* A, int a_dtype, const void* W, int w_dtype, void* C, int c_dtype,
                            const int* sorted, const int* tiles, int max_tiles, int N, int K, int lda, int ldc,
-                           long long w_expert_stride, int top, int gather, int scatter, int epi, cudaStream_t stream) {
+                           long long w_expert_stride, int top, int gather, int scatter, int epi, float alpha, float limit,
+                           float up_offset, cudaStream_t stream) {
+  const GluAct act{alpha, limit, up_offset};
   if (max_tiles <= 0 || N <= 0) return IE_OK;
   if (K <= 0 || top <= 0 || (epi == 1 && (N & 1))) return IE_BAD_SIZE;
   if (a_dtype == IE_BF16 && w_dtype == IE_BF16 && K % 8 == 0 && lda % 8 == 0 && w_expert_stride % 8 == 0 &&
@@ -417,14 +438,14 @@ extern "C" int ie_moe_gemm(const void* A, int a_dtype, const void* W, int w_dtyp
     dim3 grid((N + MM_BN - 1) / MM_BN, max_tiles);
     if (c_dtype == IE_BF16)
       return launch_k(moe_gemm_mma_kernel<bf16>, grid, MM_THREADS, 0, stream, (const bf16*)A, (const bf16*)W, (bf16*)C,
-                      sorted, tiles, N, K, lda, ldc, w_expert_stride, top, gather, scatter, epi);
+                      sorted, tiles, N, K, lda, ldc, w_expert_stride, top, gather, scatter, epi, act);
     return launch_k(moe_gemm_mma_kernel<float>, grid, MM_THREADS, 0, stream, (const bf16*)A, (const bf16*)W, (float*)C,
-                    sorted, tiles, N, K, lda, ldc, w_expert_stride, top, gather, scatter, epi);
+                    sorted, tiles, N, K, lda, ldc, w_expert_stride, top, gather, scatter, epi, act);
   }
   const int code = a_dtype * 4 + w_dtype * 2 + c_dtype;
 #define MG_GO(TA, TW, TC)                                                                                         \
   return launch_moe_gemm<TA, TW, TC>(A, W, C, sorted, tiles, max_tiles, N, K, lda, ldc, w_expert_stride, top, gather, \
-                                     scatter, epi, stream)
+                                     scatter, epi, act, stream)
   switch (code) {
     case 0: MG_GO(float, float, float);
     case 2: MG_GO(float, bf16, float);

@@ -71,7 +71,7 @@ def core():
     if _core is None:
         lib = load_library("core", defines=dict(BUILD_DEFINES.get("core", {})))
         P, I, F, L = c_void_p, c_int, c_float, c_longlong
-        lib.ie_embed_gather.argtypes = [P, P, I, P, I, I, I, P]
+        lib.ie_embed_gather.argtypes = [P, P, I, P, I, I, I, F, P]
         lib.ie_patch_tokens.argtypes = [P, P, P, I, P]
         lib.ie_patch_tokens.restype = c_int
         lib.ie_stamp.argtypes = [P, P]
@@ -80,7 +80,7 @@ def core():
         lib.ie_residual_add.argtypes = [P, P, I, I, I, P]
         lib.ie_rope_kv_write.argtypes = [P, P, P, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I, P]
         lib.ie_silu_mul.argtypes = [P, P, I, I, I, I, I, P]
-        lib.ie_attention_general.argtypes = [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, P, I, I, F, I, I, I, P, P]
+        lib.ie_attention_general.argtypes = [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, P, I, I, F, I, I, I, P, F, P, I, P]
         lib.ie_layernorm.argtypes = [P, P, P, P, I, P, I, P, I, I, F, P]
         lib.ie_embed_bigram.argtypes = [P, P, P, P, I, P, P, I, P, P, I, I, I, I, L, L, P]
         lib.ie_add_bias.argtypes = [P, I, P, I, I, I, I, P]
@@ -95,12 +95,12 @@ def core():
         lib.ie_outnorm_accumulate_norm.argtypes = [P, P, I, I, P, I, F, P, I, F, P, I, I, I, P]
         lib.ie_outnorm_accumulate_norm.restype = c_int
         lib.ie_causal_conv.argtypes = [P, I, P, P, I, P, L, P, I, P, P, I, I, I, I, I, I, I, P]
-        lib.ie_attention_rows.argtypes = [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P, I, P, I, I, F, I, I, I, P, P]
+        lib.ie_attention_rows.argtypes = [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P, I, P, I, I, F, I, I, I, P, F, P, I, P]
         lib.ie_linear_recurrence.argtypes = [P, I, P, I, P, P, I, P, P, P, I, P, P, I, P, P, I, I, F, F, I, I, P]
         lib.ie_rownorm_rotate_write.argtypes = [P, P, P, I, I, I, P, P, P, P, P, I, F, P, I, P, P, P, P, I, I, I, I, I, I, I, P]
-        lib.ie_moe_route.argtypes = [P, I, P, I, P, P, P, I, I, I, I, I, F, F, I, I, P]
+        lib.ie_moe_route.argtypes = [P, I, P, I, P, P, P, I, I, I, I, I, F, F, I, I, I, P]
         lib.ie_moe_sort.argtypes = [P, I, I, I, P, P, I, P]
-        lib.ie_moe_gemm.argtypes = [P, I, P, I, P, I, P, P, I, I, I, I, I, L, I, I, I, I, P]
+        lib.ie_moe_gemm.argtypes = [P, I, P, I, P, I, P, P, I, I, I, I, I, L, I, I, I, I, F, F, F, P]
         lib.ie_moe_combine.argtypes = [P, P, P, P, I, I, P, I, I, I, P]
         lib.ie_moe_tile_rows.restype = c_int
         lib.ie_head_prepare.argtypes = [P, I, I, I, I, I, P, P, I, I, I, I, I, P, I, P, I, I, I, F, P, I, I, F, P, P, P, P, I, I, I, P]
@@ -123,6 +123,8 @@ def core():
         lib.ie_mlstm_chunks.argtypes = [I, I]
         lib.ie_mlstm_state_floats.argtypes = [I, I]
         lib.ie_mlstm_state_floats.restype = c_longlong
+        lib.ie_stream_norm.argtypes = [P, P, I, I, P, P, I, P, I, I, F, P, I, P, I, I, P]
+        lib.ie_conv_qkv.argtypes = [P, I, P, P, L, I, I, P, I, P, P, P, I, F, P, I, I, F, P, P, P, P] + [I] * 11 + [P]
         lib.ie_argmax.argtypes = [P, P, I, I, L, P]
         lib.ie_repetition_penalty.argtypes = [P, P, P, I, I, L, I, P]
         lib.ie_sample.argtypes = [P, P, P, I, I, L, P]
@@ -135,7 +137,7 @@ def core():
                      "ie_heads_gemm", "ie_diff_combine", "ie_gated_residual_add", "ie_scale_rows", "ie_glu_act",
                      "ie_mingru_scan", "ie_mingru_scan_hint", "ie_scale_add_sinusoid", "ie_add_row", "ie_token_shift",
                      "ie_gate_mul", "ie_qkv_prepare", "ie_talk_combine", "ie_mlstm_scan", "ie_mlstm_finish",
-                     "ie_mlstm_chunks"):
+                     "ie_mlstm_chunks", "ie_stream_norm", "ie_conv_qkv"):
             getattr(lib, name).restype = c_int
         _core = lib
         _apply_check_limits()
@@ -143,12 +145,12 @@ def core():
 
 
 # ------------------------------------------------------------------ elementwise
-def embed_gather(ids: torch.Tensor, table: torch.Tensor, residual: torch.Tensor) -> None:
-    """residual[n] = table[ids[n]] as float32."""
+def embed_gather(ids: torch.Tensor, table: torch.Tensor, residual: torch.Tensor, scale: float = 1.0) -> None:
+    """residual[n] = table[ids[n]] * scale as float32."""
     assert ids.dtype == torch.int32 and residual.dtype == torch.float32 and table.is_contiguous()
     n, d = residual.shape
     _check(core().ie_embed_gather(_ptr(ids), _ptr(table), dtype_code(table.dtype), _ptr(residual), n, d,
-                                  table.shape[0], _stream()), "embed_gather")
+                                  table.shape[0], float(scale), _stream()), "embed_gather")
 
 
 def embed_bigram(ids: torch.Tensor, positions: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor,
@@ -291,7 +293,8 @@ def attention_general(q: torch.Tensor, out: torch.Tensor, kpool: torch.Tensor, v
                       n_kv_heads: int, head_dim: int, page_size: int, window: int | None, scale: float,
                       score_bias: torch.Tensor | None = None, head_scale: torch.Tensor | None = None,
                       v_head_dim: int | None = None, keep_first: int = 0, out_scale: float = 1.0, chunk: int = 0,
-                      n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None) -> None:
+                      n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None,
+                      softcap: float = 0.0, gate: torch.Tensor | None = None) -> None:
     """Paged causal attention in float32 arithmetic.  ``score_bias`` (float32 [n_heads, D], contiguous) is added to
     the scaled score of a query at position p and a key at position j as ``score_bias[head, min(p - j, D - 1)]``.
     ``head_scale`` (float32 [n_heads]) multiplies the score of its head beside ``scale``.  ``v_head_dim``: head size of
@@ -300,7 +303,9 @@ def attention_general(q: torch.Tensor, out: torch.Tensor, kpool: torch.Tensor, v
     its own chunk of that many positions.  ``n_v_heads``: heads of the value pool when several key heads share a value
     head; ``v_row``: elements between value rows when the values are the first dimensions of the key rows (one pool).
     ``sink`` (float32 [n_heads]): the softmax's denominator of head h also holds exp(sink[h]), a term without a key or
-    a value that ``scale`` does not touch."""
+    a value that ``scale`` does not touch.  ``softcap`` > 0: a scaled score s becomes softcap * tanh(s / softcap).
+    ``gate`` ([tokens, n_heads], of q's type): head h's output is multiplied by sigmoid(gate[:, h])."""
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (q.shape[0], n_heads))
     assert sink is None or (sink.dtype is torch.float32 and sink.is_contiguous() and sink.shape == (n_heads,))
     assert q.stride(1) == 1 and out.stride(1) == 1 and kpool.dtype == q.dtype == out.dtype
     assert block_table.dtype == torch.int32 and block_table.stride(1) == 1
@@ -315,7 +320,8 @@ def attention_general(q: torch.Tensor, out: torch.Tensor, kpool: torch.Tensor, v
                                        dtype_code(q.dtype), _ptr(score_bias),
                                        score_bias.shape[1] if score_bias is not None else 0, _ptr(head_scale),
                                        int(v_head_dim or head_dim), int(keep_first or 0), float(out_scale),
-                                       int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), _ptr(sink), _stream()),
+                                       int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), _ptr(sink), float(softcap),
+                                       _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
            f"attention_general(head_dim={head_dim}, heads={n_heads}/{n_kv_heads})")
 
 
@@ -324,10 +330,12 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, kpool: torch.Tensor, vpoo
                    n_kv_heads: int, head_dim: int, page_size: int, window: int | None, scale: float,
                    score_bias: torch.Tensor | None = None, head_scale: torch.Tensor | None = None,
                    v_head_dim: int | None = None, keep_first: int = 0, out_scale: float = 1.0, chunk: int = 0,
-                   n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None) -> None:
+                   n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None,
+                   softcap: float = 0.0, gate: torch.Tensor | None = None) -> None:
     """``attention_general`` for the requests of the step that bring at most ``max_rows`` (token, head-in-group) rows
     (decode tokens, as a rule): a block per (token, query head) whose warps split the visible keys.  Rows of requests
     that bring more are left untouched (the tile kernel's, with a work list of those requests)."""
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (q.shape[0], n_heads))
     assert q.stride(1) == 1 and out.stride(1) == 1 and kpool.dtype == q.dtype == out.dtype
     assert block_table.dtype == torch.int32 and block_table.stride(1) == 1
     if score_bias is not None:
@@ -340,7 +348,8 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, kpool: torch.Tensor, vpoo
                                     float(scale), dtype_code(q.dtype), _ptr(score_bias),
                                     score_bias.shape[1] if score_bias is not None else 0, _ptr(head_scale),
                                     int(v_head_dim or head_dim), int(keep_first or 0), float(out_scale),
-                                    int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), _ptr(sink), _stream()),
+                                    int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), _ptr(sink), float(softcap),
+                                    _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
            f"attention_rows(head_dim={head_dim}, heads={n_heads}/{n_kv_heads})")
 
 
@@ -720,17 +729,20 @@ def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
     return -(-n_pairs // moe_tile_rows()) + min(n_experts, n_pairs)
 
 
-ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1}
+ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1, "softmax": 2}
+GROUP_SCORES = {"top2_sum": 0, "max": 1}
 
 
 def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, ids: torch.Tensor, weights: torch.Tensor,
               gate: torch.Tensor | None, n_experts: int, top: int, n_groups: int, keep_groups: int, route_scale: float,
-              weight_eps: float, gate_col: int = -1, score: str = "sigmoid") -> None:
+              weight_eps: float, gate_col: int = -1, score: str = "sigmoid", group_score: str = "top2_sum") -> None:
     """Per token, from float32 router ``logits`` [n, >= n_experts]: the chosen experts ``ids`` int32 [n, top] and their
     ``weights`` float32 [n, top]; ``gate`` float32 [n] = sigmoid(logits[:, gate_col]) (the shared expert's).  ``score``
     "sigmoid": sigmoid scores, ``correction`` added for the choice only, weights the chosen scores over their sum.
     "softmax_top": ``correction`` is a bias of the logits themselves, the largest ``top`` are chosen and their weights
-    are the softmax over the chosen logits alone (times ``route_scale``)."""
+    are the softmax over the chosen logits alone (times ``route_scale``).  "softmax": as "sigmoid" with the softmax over
+    all experts as the scores.  ``group_score``: a group's score is the sum of its two largest choice scores
+    ("top2_sum") or the largest one ("max")."""
     n = logits.shape[0]
     assert logits.dtype is torch.float32 and logits.stride(1) == 1 and ids.dtype is torch.int32 and ids.is_contiguous()
     assert weights.dtype is torch.float32 and weights.is_contiguous() and ids.shape == weights.shape == (n, top)
@@ -738,7 +750,7 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, ids: torch.
     _check(core().ie_moe_route(_ptr(logits), logits.stride(0), _ptr(correction),
                                dtype_code(correction.dtype) if correction is not None else IE_F32, _ptr(ids),
                                _ptr(weights), _ptr(gate), n, n_experts, top, n_groups, keep_groups, float(route_scale),
-                               float(weight_eps), int(gate_col), ROUTE_SCORES[score], _stream()), f"moe_route(experts={n_experts}, top={top})")
+                               float(weight_eps), int(gate_col), ROUTE_SCORES[score], GROUP_SCORES[group_score], _stream()), f"moe_route(experts={n_experts}, top={top})")
 
 
 def moe_sort(ids: torch.Tensor, n_experts: int, sorted_pairs: torch.Tensor, tiles: torch.Tensor) -> None:
@@ -752,15 +764,19 @@ def moe_sort(ids: torch.Tensor, n_experts: int, sorted_pairs: torch.Tensor, tile
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, sorted_pairs: torch.Tensor, tiles: torch.Tensor,
-             top: int, gather: bool, scatter: bool, epi: str = "store") -> None:
+             top: int, gather: bool, scatter: bool, epi: str = "store", act: tuple[float, float, float] | None = None) -> None:
     """The grouped product over the tiles of ``moe_sort``: ``w`` [experts, N, K]; ``gather``: a pair's row of ``a`` is
     its token's (pair // top), else its sorted position; ``scatter``: its row of ``c`` is the pair's index, else its
-    sorted position; ``epi`` "silu_mul": w's rows alternate gate, up and c is N / 2 wide."""
+    sorted position; ``epi`` "silu_mul": w's rows alternate gate, up and c, N / 2 wide, takes the gated activation: silu(g) *
+    u, or with ``act`` = (alpha, limit, up_offset) g' sigmoid(alpha g') * (u' + up_offset), g' = min(g, limit), u' = u
+    clamped to [-limit, limit]."""
+    alpha, limit, up_offset = act if act is not None else (1.0, float("inf"), 0.0)
     _, n, k = w.shape
     assert w.is_contiguous() and a.stride(1) == 1 and c.stride(1) == 1 and a.shape[1] == k
     _check(core().ie_moe_gemm(_ptr(a), dtype_code(a.dtype), _ptr(w), dtype_code(w.dtype), _ptr(c), dtype_code(c.dtype),
                               _ptr(sorted_pairs), _ptr(tiles), tiles.shape[0], n, k, a.stride(0), c.stride(0), n * k, top,
-                              1 if gather else 0, 1 if scatter else 0, {"store": 0, "silu_mul": 1}[epi], _stream()),
+                              1 if gather else 0, 1 if scatter else 0, {"store": 0, "silu_mul": 1}[epi], float(alpha), float(limit),
+                              float(up_offset), _stream()),
            f"moe_gemm(n={n}, k={k}, {epi})")
 
 
@@ -775,6 +791,70 @@ def moe_combine(y: torch.Tensor, weights: torch.Tensor, gate: torch.Tensor | Non
                                  dtype_code(shared_out.dtype) if shared_out is not None else IE_F32,
                                  shared_out.stride(0) if shared_out is not None else 0, _ptr(out), n, d, top, _stream()),
            "moe_combine")
+
+
+# ------------------------------------------------- a scaled sum into the stream, convolved queries, keys and values
+def stream_norm(residual: torch.Tensor, y: torch.Tensor | None, scale: torch.Tensor | None, weights: torch.Tensor | None,
+                gain: torch.Tensor | None, groups: int, eps: float, out: torch.Tensor | None,
+                row_index: torch.Tensor | None = None) -> None:
+    """residual (float32 [n, d]) += scale * y, coordinate by coordinate (``scale`` float32 [d], None: 1; ``y`` None:
+    nothing is added), and ``out`` (None: the sum alone) = the RMS norm of the new rows in ``groups`` equal consecutive
+    parts, each by itself, times ``gain``.  With ``weights`` (float32 [n, top]) ``y`` is [n * top, d] and a row's summand
+    is ``sum_r weights[n, r] * y[n * top + r]``.  With ``row_index`` only those rows are normed and the residual keeps
+    its values."""
+    n, d = residual.shape
+    top = weights.shape[1] if weights is not None else 1
+    assert residual.dtype is torch.float32 and residual.is_contiguous()
+    assert y is None or (y.stride(1) == 1 and y.shape == (n * top, d))
+    assert scale is None or (scale.dtype is torch.float32 and scale.is_contiguous() and scale.shape == (d,))
+    assert weights is None or (weights.dtype is torch.float32 and weights.is_contiguous() and weights.shape == (n, top))
+    assert out is None or (out.is_contiguous() and out.shape[1] == d and gain.is_contiguous() and gain.shape == (d,))
+    assert row_index is not None or out is None or out.shape[0] == n
+    _check(core().ie_stream_norm(_ptr(residual), _ptr(y), dtype_code(y.dtype) if y is not None else IE_F32,
+                                 y.stride(0) if y is not None else d, _ptr(scale), _ptr(weights), top, _ptr(gain),
+                                 dtype_code(gain.dtype) if gain is not None else IE_F32, int(groups), float(eps), _ptr(out),
+                                 dtype_code(out.dtype) if out is not None else IE_F32, _ptr(row_index),
+                                 out.shape[0] if out is not None else n, d, _stream()), f"stream_norm(groups={groups})")
+
+
+V_MODES = {None: 0, "keep": 1, "mix": 2}
+
+
+def conv_qkv(x: torch.Tensor, weight: torch.Tensor | None, state: torch.Tensor | None, q_out: torch.Tensor,
+             kpool: torch.Tensor | None, vpool: torch.Tensor | None, positions: torch.Tensor,
+             slot_mapping: torch.Tensor | None, q_start: torch.Tensor, slots: torch.Tensor, n_requests: int, n_heads: int,
+             n_kv_heads: int, head_dim: int, v_head_dim: int, k_col: int, v_col: int, page_size: int,
+             inv_freq: torch.Tensor | None = None, rot_dims: int = 0, neighbours: bool = True, mult: float = 1.0,
+             v_kept: torch.Tensor | None = None, v_mode: str | None = None, lam: float = 0.0, write_state: bool = True,
+             max_q_len: int | None = None) -> None:
+    """From the raw projections ``x`` [n, channels] (queries, keys from column ``k_col``, values from ``v_col``) to what
+    attention reads: a causal convolution over time per channel (``weight`` float32 [taps, channels], its last row
+    multiplies the current token; None: none) whose last inputs are ``state`` [slots, taps - 1, channels] of x's type; a
+    rotation of the first ``rot_dims`` dimensions of every query and key head (``inv_freq`` float64 [rot_dims / 2], sine
+    and cosine times ``mult``); values written to ``v_kept`` [n, kv heads * v_head_dim] (``v_mode`` "keep") or blended
+    with it, ``(1 - lam) v + lam v_kept`` ("mix").  Queries go to ``q_out``, keys and values to the tokens' slots of the
+    pools [pages, kv heads, page_size, size]."""
+    n, channels = x.shape
+    taps = weight.shape[0] if weight is not None else 1
+    assert x.stride(1) == 1 and q_out.stride(1) == 1 and q_out.dtype == x.dtype and q_out.shape == (n, n_heads * head_dim)
+    assert q_out.data_ptr() != x.data_ptr(), "the convolution reads earlier rows of its input after writing its output"
+    assert weight is None or (weight.dtype is torch.float32 and weight.is_contiguous() and weight.shape == (taps, channels))
+    assert taps <= CONV_MAX_TAPS
+    assert taps == 1 or (state is not None and state.dtype == x.dtype and state.shape[1:] == (taps - 1, channels)
+                         and state.stride(2) == 1 and state.stride(1) == channels)
+    for pool, size in ((kpool, head_dim), (vpool, v_head_dim)):
+        assert pool is None or (pool.dtype == x.dtype and pool.is_contiguous() and pool.shape[1:] == (n_kv_heads, page_size, size))
+    assert v_mode is None or (v_kept is not None and v_kept.dtype == x.dtype and v_kept.is_contiguous()
+                              and v_kept.shape == (n, n_kv_heads * v_head_dim))
+    assert inv_freq is None or (inv_freq.dtype is torch.float64 and inv_freq.is_contiguous() and inv_freq.numel() * 2 >= rot_dims)
+    _check(core().ie_conv_qkv(_ptr(x), x.stride(0), _ptr(weight), _ptr(state) if taps > 1 else None,
+                              state.stride(0) if taps > 1 else 0, channels, taps, _ptr(q_out), q_out.stride(0), _ptr(kpool),
+                              _ptr(vpool), _ptr(v_kept) if v_mode else None, V_MODES[v_mode], float(lam), _ptr(inv_freq),
+                              int(rot_dims if inv_freq is not None else 0), 1 if neighbours else 0, float(mult),
+                              _ptr(positions), _ptr(slot_mapping), _ptr(q_start), _ptr(slots), n_requests, n_heads,
+                              n_kv_heads, head_dim, v_head_dim, k_col, v_col, page_size, 1 if write_state else 0,
+                              dtype_code(x.dtype), int(max_q_len) if max_q_len else max(n, 1), _stream()),
+           f"conv_qkv(heads={n_heads}/{n_kv_heads}, {head_dim}/{v_head_dim}, taps={taps})")
 
 
 # ---------------------------------------------------------------------- sampling
@@ -903,20 +983,22 @@ def attention_wide_supports(q: torch.Tensor, out: torch.Tensor, head_dim: int, v
             and q.data_ptr() % 16 == 0 and out.data_ptr() % 4 == 0 and (v_row or v_head_dim) % 8 == 0)
 
 
-def attention_wide_library(head_dim: int, v_head_dim: int):
-    """The tensor-core attention kernel with float32 scores built for one (key, value) head size; compiled when first
-    asked for."""
-    key = (int(head_dim), int(v_head_dim))
+def attention_wide_library(head_dim: int, v_head_dim: int, capped: bool = False):
+    """The tensor-core attention kernel with float32 scores built for one (key, value) head size, with or without capped
+    scores; compiled when first asked for."""
+    key = (int(head_dim), int(v_head_dim), bool(capped))
     lib = _wide.get(key)
     if lib is None:
         defines = {"IE_AW_DK": key[0], "IE_AW_DV": key[1], **BUILD_DEFINES.get("attn_wide", {})}
-        lib = load_library(f"attn_wide_k{key[0]}_v{key[1]}", ["attention_wide.cu"], defines)
+        if capped:
+            defines["IE_AW_CAP"] = 1
+        lib = load_library(f"attn_wide_k{key[0]}_v{key[1]}" + ("_cap" if capped else ""), ["attention_wide.cu"], defines)
         P, I, F = c_void_p, c_int, c_float
-        lib.ie_attention_wide.argtypes = [P] * 9 + [I] * 8 + [F, I, I, I, P, P]
+        lib.ie_attention_wide.argtypes = [P] * 9 + [I] * 8 + [F, I, I, I, P, F, P, I, P]
         lib.ie_attention_wide.restype = c_int
         lib.ie_attention_wide_rows.restype = c_int
         lib.ie_attention_wide_keys.restype = c_int
-        lib.ie_attention_wide_small.argtypes = [P] * 7 + [I] * 9 + [F] + [I] * 5 + [P, P, P]
+        lib.ie_attention_wide_small.argtypes = [P] * 7 + [I] * 9 + [F] + [I] * 5 + [P, P, F, P, I, P]
         lib.ie_attention_wide_small.restype = c_int
         lib.ie_attention_wide_small_scratch.argtypes = [I, I, I, I]
         lib.ie_attention_wide_small_scratch.restype = c_longlong
@@ -930,7 +1012,8 @@ ATTENTION_WIDE_ROWS = 64     # (token, head-in-group) pairs of a tile of the ker
 
 def attention_wide(q, out, kpool, vpool, block_table, q_start, ctx_before, work_req, work_pair0, n_work, n_heads,
                    n_kv_heads, head_dim, page_size, window, scale, v_head_dim: int | None = None, chunk: int = 0,
-                   n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None) -> None:
+                   n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None,
+                   softcap: float = 0.0, gate: torch.Tensor | None = None) -> None:
     """Causal paged attention of prompt portions on tensor cores with float32 scores, maxima and sums, the weights to
     two bfloat16 terms: ``attention_general``'s options ``v_head_dim``, ``chunk``, ``n_v_heads`` and ``v_row`` and a
     window, for bfloat16 operands whose head sizes are multiples of 16.  The work list cuts each request's (token,
@@ -938,19 +1021,22 @@ def attention_wide(q, out, kpool, vpool, block_table, q_start, ctx_before, work_
     dv = int(v_head_dim or head_dim)
     assert attention_wide_supports(q, out, head_dim, dv, v_row) and kpool.dtype is torch.bfloat16 and vpool.dtype is torch.bfloat16
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.dtype == torch.int32 and block_table.stride(1) == 1
-    lib = attention_wide_library(head_dim, dv)
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (q.shape[0], n_heads))
+    lib = attention_wide_library(head_dim, dv, softcap > 0)
     _check(lib.ie_attention_wide(_ptr(q), _ptr(out), _ptr(kpool), _ptr(vpool), _ptr(block_table), _ptr(q_start),
                                  _ptr(ctx_before), _ptr(work_req), _ptr(work_pair0), q.stride(0), out.stride(0),
                                  block_table.stride(0), n_work, n_heads, n_kv_heads, page_size, int(window or 0),
-                                 float(scale), int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), _ptr(sink), _stream()),
+                                 float(scale), int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), _ptr(sink), float(softcap),
+                                 _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
            f"attention_wide(head_dim={head_dim}/{dv}, heads={n_heads}/{n_kv_heads})")
 
 
-def attention_wide_splits(head_dim: int, v_head_dim: int, keys: int, n_streams: int, n_sms: int | None = None) -> tuple[int, int]:
+def attention_wide_splits(head_dim: int, v_head_dim: int, keys: int, n_streams: int, n_sms: int | None = None,
+                          capped: bool = False) -> tuple[int, int]:
     """(n_splits, split_keys) for ``attention_wide_small``: ``keys`` is the longest run of keys a request may see,
     counted from the key tile's boundary below its first one; ``n_streams`` the (request tile, key head) pairs that each
     walk such a run.  Enough splits to fill the device about twice, none shorter than two key tiles."""
-    tile = int(attention_wide_library(head_dim, v_head_dim).ie_attention_wide_keys())
+    tile = int(attention_wide_library(head_dim, v_head_dim, capped).ie_attention_wide_keys())
     n_tiles = max(1, -(-int(keys) // tile))
     want = max(1, -(-2 * (n_sms or sm_count()) // max(1, n_streams)))
     n_splits = max(1, min(want, n_tiles // 2 or 1))
@@ -958,15 +1044,17 @@ def attention_wide_splits(head_dim: int, v_head_dim: int, keys: int, n_streams: 
     return -(-n_tiles // per), per * tile
 
 
-def attention_wide_small_scratch(head_dim: int, v_head_dim: int, n_requests: int, max_rows: int, n_kv_heads: int, n_splits: int) -> int:
+def attention_wide_small_scratch(head_dim: int, v_head_dim: int, n_requests: int, max_rows: int, n_kv_heads: int, n_splits: int,
+                                 capped: bool = False) -> int:
     """float32 words of scratch that ``attention_wide_small`` needs."""
-    return int(attention_wide_library(head_dim, v_head_dim).ie_attention_wide_small_scratch(n_requests, max_rows, n_kv_heads, n_splits))
+    return int(attention_wide_library(head_dim, v_head_dim, capped).ie_attention_wide_small_scratch(n_requests, max_rows, n_kv_heads, n_splits))
 
 
 def attention_wide_small(q, out, kpool, vpool, block_table, q_start, ctx_before, n_requests: int, max_rows: int, n_heads,
                          n_kv_heads, head_dim, page_size, window, scale, n_splits: int, split_keys: int,
                          scratch: torch.Tensor | None, v_head_dim: int | None = None, chunk: int = 0,
-                         n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None) -> None:
+                         n_v_heads: int | None = None, v_row: int | None = None, sink: torch.Tensor | None = None,
+                         softcap: float = 0.0, gate: torch.Tensor | None = None) -> None:
     """``attention_wide`` for the requests of the step that bring at most ``max_rows`` (token, head-in-group) rows (decode
     tokens, as a rule), without a work list: every (request, key head) is cut into ``n_splits`` runs of ``split_keys``
     keys (``attention_wide_splits``), a block each, and a second kernel merges them through ``scratch`` (float32,
@@ -974,7 +1062,8 @@ def attention_wide_small(q, out, kpool, vpool, block_table, q_start, ctx_before,
     dv = int(v_head_dim or head_dim)
     assert attention_wide_supports(q, out, head_dim, dv, v_row) and kpool.dtype is torch.bfloat16 and vpool.dtype is torch.bfloat16
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.dtype == torch.int32 and block_table.stride(1) == 1
-    lib = attention_wide_library(head_dim, dv)
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (q.shape[0], n_heads))
+    lib = attention_wide_library(head_dim, dv, softcap > 0)
     if n_splits > 1:
         need = int(lib.ie_attention_wide_small_scratch(n_requests, max_rows, n_kv_heads, n_splits))
         assert scratch is not None and scratch.dtype is torch.float32 and scratch.is_contiguous() and scratch.numel() >= need
@@ -982,7 +1071,8 @@ def attention_wide_small(q, out, kpool, vpool, block_table, q_start, ctx_before,
                                        _ptr(ctx_before), q.stride(0), out.stride(0), block_table.stride(0), n_requests,
                                        int(max_rows), n_heads, n_kv_heads, page_size, int(window or 0), float(scale),
                                        int(chunk or 0), int(n_v_heads or 0), int(v_row or 0), int(n_splits), int(split_keys),
-                                       _ptr(scratch), _ptr(sink), _stream()),
+                                       _ptr(scratch), _ptr(sink), float(softcap), _ptr(gate),
+                                       gate.stride(0) if gate is not None else 0, _stream()),
            f"attention_wide_small(head_dim={head_dim}/{dv}, heads={n_heads}/{n_kv_heads}, splits={n_splits})")
     if n_splits > 1:
         global LAUNCHES
@@ -1350,7 +1440,7 @@ def attention_tcgen05(q, out, kpool, vpool, block_table, q_start, ctx_before, wo
 CHECK_LIBRARIES = ("core", "attn_mma", "attn_tcgen05", "attn_wide", "delta_rule", "gated_delta")
 CHECK_UNITS = ("elementwise", "rowwise", "sequence", "attention_general", "attention_mma", "attention_tcgen05",
                "attention_wide", "delta_rule", "gated_delta", "headwise", "gating", "stream_shift", "headmix",
-               "matrix_memory")
+               "matrix_memory", "convqkv")
 CHECK_CODES = {1: "page id", 2: "cache slot", 3: "token id"}
 _check_limits: tuple[int, int, int] | None = None
 

@@ -1,6 +1,7 @@
-from . import attention, block, delta_rule, feedforward, gated_delta, latent, matrix_memory, model, norms, positions, recurrence, routed, talking  # noqa: F401  (register the built-in parts)
+from . import attention, block, conv_attention, delta_rule, feedforward, gated_delta, latent, matrix_memory, model, norms, positions, recurrence, routed, talking  # noqa: F401  (register the built-in parts)
 from .attention import CacheView, PagedAttention
-from .block import GatedPreNormBlock, OutputNormBlock, PreNormBlock, SandwichBlock
+from .block import GatedPreNormBlock, OutputNormBlock, PreNormBlock, SandwichBlock, ScaledPreNormBlock
+from .conv_attention import ConvAttention
 from .delta_rule import GeneralDeltaMixer
 from .feedforward import GatedMLP, PolyNormMLP
 from .gated_delta import GatedDeltaMixer
@@ -8,7 +9,7 @@ from .latent import DifferentialAttention, LatentAttention
 from .linear import Linear
 from .matrix_memory import MatrixMemory
 from .model import BigramDecoderModel, DecoderModel, PassOffsetDecoderModel, ReinjectDecoderModel
-from .norms import LayerNorm, RMSNorm
+from .norms import GroupedRMSNorm, LayerNorm, RMSNorm, ScaledDelta
 from .positions import BucketedBias, NoPosition, PartialRotation, Rotary, RotaryPairs, distance_bucket, rotary_inv_freq, rotary_tables
 from .recurrence import GatedLinearRecurrence, MinGRU, ParallelMixer
 from .registry import (

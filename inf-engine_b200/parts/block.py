@@ -1,14 +1,18 @@
 """Residual blocks.  The pre-norm block: ``x += mixer(norm(x)); x += ff(norm(x))``
 (engine/llama_block.py:50-62); beside it a block that norms its sublayers' outputs, a pre-norm block with gates per
-coordinate, and a block with a norm before and after each sublayer whose mixer may read shifted inputs.  The sums are folded into the norm that follows
+coordinate, and a block with a norm before and after each sublayer whose mixer may read shifted inputs, and a pre-norm block whose
+sublayers' results take a multiplier per coordinate.  The sums are folded into the norm that follows
 them: a block hands on the residual and a delta that is not added yet.  A block
 whose spec has no feed-forward is the first half alone."""
 
 from __future__ import annotations
 
+import torch
+
 from .. import kernels
 from ..weights.loader import ExpectedTensor
 from .linear import Linear
+from .norms import ScaledDelta, add_pending
 from .registry import (
     build_feedforward,
     build_mixer,
@@ -56,7 +60,7 @@ class PreNormBlock:
         ff_fuses = self.feedforward is not None and _fuses(self.feedforward, n, self.ff_norm)
         if _fuses(self.mixer, n, self.mixer_norm):
             if pending is not None:
-                kernels.residual_add(residual, pending)
+                add_pending(residual, pending)
                 ctx.handover = None
             ctx.upcoming_norm = self.ff_norm if ff_fuses else None
             self.mixer.forward_fused(residual, self.mixer_norm, ctx, cache)
@@ -128,7 +132,7 @@ class OutputNormBlock:
         ctx.handover = None
         ctx.upcoming_norm = None
         if pending is not None:
-            kernels.residual_add(residual, pending)
+            add_pending(residual, pending)
             ctx.residual_cast = None
         a = self.mixer.forward(self._input(residual, ctx), ctx, cache)
         last = getattr(ctx, "last_block", False)
@@ -284,6 +288,60 @@ class SandwichBlock:
             h = self.ff_norm.add_norm(residual, None)
         self.ff_out_norm.accumulate(residual, self.feedforward.forward(h, ctx))
         return residual, None
+
+
+@register_block("scaled_prenorm")
+class ScaledPreNormBlock:
+    """``x += c * s1 * mixer(norm1(x))``, then ``x += c * s2 * ff(norm2(x))``: a pre-norm block whose sublayers' results
+    are multiplied by a constant (``residual_mult``) and by a learned number per coordinate (``mixer_scale`` /
+    ``ff_scale``) before the sum.  Constant and vector are one float32 vector, formed once; the product, the sum into
+    the float32 residual and the norm that comes next are one kernel (a norm that takes a ``ScaledDelta``), which for a
+    mixture of experts also forms the weighted sum of the chosen experts' results."""
+
+    @staticmethod
+    def expected_tensors(spec):
+        d = spec.mixer_norm.size
+        out = PreNormBlock.expected_tensors(spec)
+        if spec.mixer_scale is not None:
+            out[spec.mixer_scale] = ExpectedTensor((d,), init="gain")
+        if spec.feedforward is not None and spec.ff_scale is not None:
+            out[spec.ff_scale] = ExpectedTensor((d,), init="gain")
+        return out
+
+    def __init__(self, spec, tensors, rt):
+        self.spec = spec
+        self.mixer_norm = build_norm(spec.mixer_norm, tensors, rt)
+        self.mixer = build_mixer(spec.mixer, tensors, rt)
+        has_ff = spec.feedforward is not None
+        self.ff_norm = build_norm(spec.ff_norm, tensors, rt) if has_ff else None
+        self.feedforward = build_feedforward(spec.feedforward, tensors, rt) if has_ff else None
+
+        def scale(name):
+            if name is None and spec.residual_mult == 1.0:
+                return None
+            d = spec.mixer_norm.size
+            s = tensors[name].float() if name is not None else torch.ones(d, dtype=torch.float32, device=rt.device)
+            return (s * float(spec.residual_mult)).contiguous()
+
+        self.mixer_scale = scale(spec.mixer_scale)
+        self.ff_scale = scale(spec.ff_scale) if has_ff else None
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(p, "graph_safe", False) for p in (self.mixer, self.feedforward) if p is not None)
+
+    def forward(self, residual, pending, ctx, cache):
+        ctx.handover = None
+        ctx.upcoming_norm = None
+        ctx.residual_cast = None
+        h = self.mixer_norm.add_norm(residual, pending)
+        pending = ScaledDelta(self.mixer.forward(h, ctx, cache), self.mixer_scale)
+        if self.feedforward is None:
+            return residual, pending
+        h = self.ff_norm.add_norm(residual, pending)
+        unsummed = getattr(self.feedforward, "forward_unsummed", None)
+        y, weights = unsummed(h, ctx) if unsummed is not None else (self.feedforward.forward(h, ctx), None)
+        return residual, ScaledDelta(y, self.ff_scale, weights)
 
 
 def _fuses(part, n_tokens: int, norm) -> bool:

@@ -36,21 +36,24 @@ WIDE_SMALL_MIN_GROUP = 4      # query heads a key head from which decode tokens 
 
 def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int,
                    scale: float, chunk: int | None, n_v_heads: int | None = None, v_row: int | None = None,
-                   window: int | None = None, sink: torch.Tensor | None = None) -> None:
+                   window: int | None = None, sink: torch.Tensor | None = None, softcap: float = 0.0,
+                   gate: torch.Tensor | None = None) -> None:
     """Causal attention of the step's queries over the paged keys with float32 scores, maxima, weights and sums.
     Requests of at most ``SMALL_REQUEST_TOKENS`` tokens (decode tokens): a block per (token, head) whose warps split the
     keys, or, in bfloat16 storage with head sizes that are multiples of 16 and several query heads a key head, the
     tensor-core kernel with the keys split over blocks (every key row is then loaded once for all those heads).  The
     others (prompt portions), through a work list: the tensor-core kernel under the same conditions, else the float32
     tile kernel.  ``window``: a query sees itself and the window - 1 keys before it.  ``sink`` (float32 [n_heads]): a
-    term exp(sink_h) without key or value in the denominator of head h."""
+    term exp(sink_h) without key or value in the denominator of head h.  ``softcap`` > 0: scores pass softcap *
+    tanh(s / softcap).  ``gate`` ([tokens, n_heads]): head h's output times sigmoid(gate_h)."""
     group = n_heads // n_kv_heads
     max_rows = SMALL_REQUEST_TOKENS * group
     if ctx.max_q_len <= SMALL_REQUEST_TOKENS:
         n_small = ctx.n_requests
     else:
         n_small = sum(1 for n in ctx.host["q_lens"] if n <= SMALL_REQUEST_TOKENS)
-    extra = dict(v_head_dim=v_head_dim, chunk=chunk or 0, n_v_heads=n_v_heads, v_row=v_row, sink=sink)
+    extra = dict(v_head_dim=v_head_dim, chunk=chunk or 0, n_v_heads=n_v_heads, v_row=v_row, sink=sink, softcap=softcap,
+                 gate=gate)
     wide = (kpool.dtype is torch.bfloat16 and kernels.attention_wide_supports(q, out, head_dim, v_head_dim, v_row)
             and kpool.data_ptr() % 16 == 0 and vpool.data_ptr() % 16 == 0)
     if n_small:
@@ -61,8 +64,9 @@ def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: i
             if window:
                 keys = min(keys, window + SMALL_REQUEST_TOKENS)
             n_splits, split_keys = kernels.attention_wide_splits(head_dim, v_head_dim, keys + 64,
-                                                                  ctx.n_requests * -(-max_rows // rows) * n_kv_heads)
-            words = kernels.attention_wide_small_scratch(head_dim, v_head_dim, ctx.n_requests, max_rows, n_kv_heads, n_splits)
+                                                                  ctx.n_requests * -(-max_rows // rows) * n_kv_heads, capped=softcap > 0)
+            words = kernels.attention_wide_small_scratch(head_dim, v_head_dim, ctx.n_requests, max_rows, n_kv_heads, n_splits,
+                                                         capped=softcap > 0)
             scratch = ctx.rt.ws.take("attn_wide_scratch", (words,), torch.float32) if words else None
             kernels.attention_wide_small(q, out, kpool, vpool, kvctx.block_table, ctx.q_start, ctx.ctx_before, ctx.n_requests,
                                          max_rows, n_heads, n_kv_heads, head_dim, ctx.page_size, window, scale, n_splits,

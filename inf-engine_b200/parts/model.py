@@ -12,6 +12,7 @@ from .. import kernels
 from ..cache.manager import CacheManager, CacheRequirement
 from .attention import CacheView
 from .linear import Linear, stream_normed
+from .norms import add_pending
 from ..weights.loader import ExpectedTensor
 from .registry import block_class, build_block, build_norm, norm_class, register_model
 
@@ -80,8 +81,11 @@ class DecoderModel:
     # ---------------------------------------------------------------- forward
     def embed(self, ctx) -> torch.Tensor:
         """The float32 residual stream [n_tokens, hidden] that the first block meets."""
+        return self._embedding_rows(ctx, self.spec.embedding_scale)
+
+    def _embedding_rows(self, ctx, scale: float) -> torch.Tensor:
         residual = self.rt.ws.take("residual", (ctx.n_tokens, self.spec.hidden), torch.float32)
-        kernels.embed_gather(ctx.token_ids, self.embedding, residual)
+        kernels.embed_gather(ctx.token_ids, self.embedding, residual, scale)
         return residual
 
     def before_entry(self, i: int, residual, pending, ctx):
@@ -122,7 +126,7 @@ class DecoderModel:
         if self.head.streams(m, normed=True) and hasattr(self.final_norm, "fusable_rms"):
             # final norm on the gathered rows inside the head product
             if pending is not None:
-                kernels.residual_add(residual, pending)
+                add_pending(residual, pending)
                 ctx.handover = None
             if m == n and getattr(ctx, "handover", None) is not None:
                 # every row is wanted (a decode step): the last block may have prepared the final norm's input
@@ -151,6 +155,8 @@ class BigramDecoderModel(DecoderModel):
         super().__init__(spec, tensors, rt)
         if spec.bigram_buckets <= 0:
             raise ValueError("a hashed bigram embedding needs a positive number of buckets")
+        if spec.embedding_scale != 1.0:
+            raise NotImplementedError("a hashed bigram embedding with a scaled token embedding is not built")
         self.bigram = tensors[spec.bigram].to(self.embedding.dtype)
         self._prev_token: torch.Tensor | None = None
 
@@ -189,15 +195,15 @@ class ReinjectDecoderModel(DecoderModel):
     def embed(self, ctx) -> torch.Tensor:
         residual = super().embed(ctx)
         self._embedded = self.rt.ws.take("embedded", tuple(residual.shape), torch.float32) if self.reinject else None
-        if self.spec.embedding_scale != 1.0 or self._embedded is not None:
-            kernels.scale_rows(residual, self.spec.embedding_scale, self._embedded)
+        if self._embedded is not None:
+            kernels.scale_rows(residual, 1.0, self._embedded)
         return residual
 
     def before_entry(self, i: int, residual, pending, ctx):
         if i not in self.reinject:
             return residual, pending
         if pending is not None:
-            kernels.residual_add(residual, pending)
+            add_pending(residual, pending)
         kernels.residual_add(residual, self._embedded)
         ctx.handover = None
         ctx.residual_cast = None
@@ -229,12 +235,11 @@ class PassOffsetDecoderModel(DecoderModel):
             self.offsets[int(entry)] = tensors[spec.pass_offsets][int(row)].contiguous()
 
     def embed(self, ctx) -> torch.Tensor:
-        residual = super().embed(ctx)
         s = self.spec
-        if s.sinusoid_base > 0:
-            kernels.scale_add_sinusoid(residual, ctx.positions, s.embedding_scale, s.sinusoid_base)
-        elif s.embedding_scale != 1.0:
-            kernels.scale_rows(residual, s.embedding_scale)
+        if s.sinusoid_base <= 0:
+            return super().embed(ctx)
+        residual = self._embedding_rows(ctx, 1.0)
+        kernels.scale_add_sinusoid(residual, ctx.positions, s.embedding_scale, s.sinusoid_base)
         return residual
 
     def before_entry(self, i: int, residual, pending, ctx):
@@ -242,7 +247,7 @@ class PassOffsetDecoderModel(DecoderModel):
         if row is None:
             return residual, pending
         if pending is not None:
-            kernels.residual_add(residual, pending)
+            add_pending(residual, pending)
         kernels.add_row(residual, row)
         ctx.handover = None
         ctx.residual_cast = None

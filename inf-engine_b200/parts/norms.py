@@ -5,6 +5,8 @@ that precedes it in a pre-norm block (engine/llama_block.py:53-62).  With
 (formed once, in float32); with ``scalar`` the stored tensor is a single number that multiplies every coordinate.
 ``accumulate`` is the norm of a block that norms its
 sublayers' OUTPUTS: the normed rows are added into the residual.
+``GroupedRMSNorm`` norms each of several equal consecutive parts of the row by itself, and takes a summand that carries
+a multiplier per coordinate or is a mixture of experts not summed up yet (``ScaledDelta``) in the same kernel.
 LayerNorm: ``(x - mean) / sqrt(variance + eps) * weight + bias`` with the variance
 the mean of the squared deviations, the same way."""
 
@@ -15,6 +17,32 @@ import torch
 from .. import kernels
 from ..weights.loader import ExpectedTensor
 from .registry import register_norm
+
+
+class ScaledDelta:
+    """A summand of the residual stream that is not added yet: ``scale * y`` with ``scale`` float32 [d] (None: 1), or
+    ``scale * sum_r weights[n, r] * y[n * top + r]`` with ``weights`` float32 [n, top]."""
+
+    __slots__ = ("y", "scale", "weights")
+
+    def __init__(self, y: torch.Tensor, scale: torch.Tensor | None = None, weights: torch.Tensor | None = None):
+        self.y, self.scale, self.weights = y, scale, weights
+
+
+def add_pending(residual: torch.Tensor, pending) -> None:
+    """residual += pending, a tensor or a ``ScaledDelta``."""
+    if isinstance(pending, ScaledDelta):
+        kernels.stream_norm(residual, pending.y, pending.scale, pending.weights, None, 1, 0.0, None)
+    else:
+        kernels.residual_add(residual, pending)
+
+
+def plain_delta(residual: torch.Tensor, delta):
+    """``delta`` as the norms that take a tensor or nothing want it: a ``ScaledDelta`` is added here and now."""
+    if isinstance(delta, ScaledDelta):
+        add_pending(residual, delta)
+        return None
+    return delta
 
 
 @register_norm("rmsnorm")
@@ -55,14 +83,48 @@ class RMSNorm:
 
     def add_norm(self, residual: torch.Tensor, delta: torch.Tensor | None, out_name: str = "normed") -> torch.Tensor:
         out = self.rt.ws.take(out_name, tuple(residual.shape), self.rt.act_dtype)
-        kernels.rmsnorm(residual, delta, self.gain, out, self.eps)
+        kernels.rmsnorm(residual, plain_delta(residual, delta), self.gain, out, self.eps)
         return out
 
     def gather_norm(self, residual: torch.Tensor, delta: torch.Tensor | None, row_index: torch.Tensor,
                     n_rows: int, out_name: str = "normed_rows") -> torch.Tensor:
         out = self.rt.ws.take(out_name, (n_rows, self.size), self.rt.act_dtype)
-        kernels.rmsnorm(residual, delta, self.gain, out, self.eps, row_index=row_index)
+        kernels.rmsnorm(residual, plain_delta(residual, delta), self.gain, out, self.eps, row_index=row_index)
         return out
+
+
+@register_norm("grouped_rmsnorm")
+class GroupedRMSNorm:
+    """RMS norm of each of ``groups`` equal consecutive parts of the row by itself; the whole times the gain (and a
+    constant, formed into the gain once)."""
+
+    @staticmethod
+    def expected_tensors(spec):
+        return {spec.weight: ExpectedTensor((spec.size,), init="gain")}
+
+    def __init__(self, spec, tensors, rt):
+        if spec.groups <= 0 or spec.size % spec.groups:
+            raise ValueError(f"a row of {spec.size} does not split into {spec.groups} equal parts")
+        self.spec = spec
+        self.rt = rt
+        self.gain = tensors[spec.weight].contiguous()
+        if spec.out_scale != 1.0:
+            self.gain = (self.gain.float() * spec.out_scale).contiguous()
+        self.eps = float(spec.eps)
+        self.size = spec.size
+        self.groups = int(spec.groups)
+
+    def _norm(self, residual, delta, out, row_index=None):
+        d = delta if isinstance(delta, ScaledDelta) else ScaledDelta(delta)
+        kernels.stream_norm(residual, d.y, d.scale, d.weights, self.gain, self.groups, self.eps, out, row_index)
+        return out
+
+    def add_norm(self, residual: torch.Tensor, delta, out_name: str = "normed") -> torch.Tensor:
+        return self._norm(residual, delta, self.rt.ws.take(out_name, tuple(residual.shape), self.rt.act_dtype))
+
+    def gather_norm(self, residual: torch.Tensor, delta, row_index: torch.Tensor, n_rows: int,
+                    out_name: str = "normed_rows") -> torch.Tensor:
+        return self._norm(residual, delta, self.rt.ws.take(out_name, (n_rows, self.size), self.rt.act_dtype), row_index)
 
 
 @register_norm("layernorm")
@@ -84,11 +146,11 @@ class LayerNorm:
 
     def add_norm(self, residual: torch.Tensor, delta: torch.Tensor | None, out_name: str = "normed") -> torch.Tensor:
         out = self.rt.ws.take(out_name, tuple(residual.shape), self.rt.act_dtype)
-        kernels.layernorm(residual, delta, self.weight, self.bias, out, self.eps)
+        kernels.layernorm(residual, plain_delta(residual, delta), self.weight, self.bias, out, self.eps)
         return out
 
     def gather_norm(self, residual: torch.Tensor, delta: torch.Tensor | None, row_index: torch.Tensor,
                     n_rows: int, out_name: str = "normed_rows") -> torch.Tensor:
         out = self.rt.ws.take(out_name, (n_rows, self.size), self.rt.act_dtype)
-        kernels.layernorm(residual, delta, self.weight, self.bias, out, self.eps, row_index=row_index)
+        kernels.layernorm(residual, plain_delta(residual, delta), self.weight, self.bias, out, self.eps, row_index=row_index)
         return out

@@ -1,5 +1,5 @@
-"""A mixture of gated feed-forward experts, chosen and run on the device: a sigmoid router with groups, or (``score``
-"softmax_top") the largest logits plus a bias, weighted by the softmax over the chosen logits alone.
+"""A mixture of gated feed-forward experts, chosen and run on the device: a sigmoid or softmax router with groups, or
+(``score`` "softmax_top") the largest logits plus a bias, weighted by the softmax over the chosen logits alone.
 
 Per token, with x the part's input (``RoutedExpertsSpec`` states the rule in full):
 
@@ -60,6 +60,13 @@ class RoutedExperts:
             raise ValueError("a router whose weights are the softmax over the chosen logits has no groups and no correction")
         if spec.score != "softmax_top" and spec.router_bias is not None:
             raise ValueError("a bias of the router's logits belongs to the softmax over the chosen logits")
+        if spec.group_score not in kernels.GROUP_SCORES:
+            raise ValueError(f"group score {spec.group_score!r} is not built (known: {', '.join(kernels.GROUP_SCORES)})")
+        if spec.activation not in kernels.GLU_KINDS:
+            raise ValueError(f"activation {spec.activation!r} is not built (known: {sorted(kernels.GLU_KINDS)})")
+        # the activation in the first product's epilogue: (alpha, limit, offset of the up branch)
+        self.act = (1.0, float("inf"), spec.up_offset) if spec.activation == "silu" \
+            else (spec.act_alpha, spec.act_limit, spec.up_offset)
         self.spec = spec
         self.rt = rt
         names = [f"{spec.expert_prefix}{e}." for e in range(E)]
@@ -78,7 +85,8 @@ class RoutedExperts:
             self.correction = tensors[spec.router_bias].contiguous()      # the route kernel adds it to the logits
         self.shared = GatedMLP(spec.shared, tensors, rt) if spec.shared is not None else None
 
-    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+    def _run_experts(self, x: torch.Tensor):
+        """(the chosen experts' results [n * top, hidden] float32, their weights [n, top], the shared expert's gate)."""
         s, rt, ws = self.spec, self.rt, self.rt.ws
         n, E, top = x.shape[0], s.n_experts, s.top
         n_pairs = n * top
@@ -89,15 +97,30 @@ class RoutedExperts:
         weights = ws.take("moe_weights", (n, top), torch.float32)
         gate = ws.take("moe_gate", (n,), torch.float32) if self.shared is not None else None
         kernels.moe_route(logits, self.correction, ids, weights, gate, E, top, s.n_groups, s.keep_groups, s.route_scale,
-                          s.weight_eps, gate_col=E if self.shared is not None else -1, score=s.score)
+                          s.weight_eps, gate_col=E if self.shared is not None else -1, score=s.score, group_score=s.group_score)
         sorted_pairs = ws.take("moe_sorted", (n_pairs,), torch.int32)
         tiles = ws.take("moe_tiles", (kernels.moe_max_tiles(n_pairs, E), 4), torch.int32)
         kernels.moe_sort(ids, E, sorted_pairs, tiles)
         hidden = ws.take("moe_hidden", (n_pairs, s.intermediate), rt.act_dtype)       # in sorted order
-        kernels.moe_gemm(x, self.gate_up, hidden, sorted_pairs, tiles, top, gather=True, scatter=False, epi="silu_mul")
+        kernels.moe_gemm(x, self.gate_up, hidden, sorted_pairs, tiles, top, gather=True, scatter=False, epi="silu_mul",
+                         act=self.act)
         y = ws.take("moe_pairs_out", (n_pairs, s.hidden), torch.float32)               # in the pairs' own order
         kernels.moe_gemm(hidden, self.down, y, sorted_pairs, tiles, top, gather=False, scatter=True)
+        return y, weights, gate
+
+    @property
+    def forward_unsummed(self):
+        """``(y, weights)`` for a caller that forms ``sum_r weights[n, r] * y[n * top + r]`` itself, or None where there
+        is more to the result than that sum."""
+        return self._unsummed if self.shared is None else None
+
+    def _unsummed(self, x: torch.Tensor, ctx):
+        y, weights, _ = self._run_experts(x)
+        return y, weights
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        y, weights, gate = self._run_experts(x)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
-        out = ws.take("moe_out", (n, s.hidden), torch.float32)
+        out = self.rt.ws.take("moe_out", (x.shape[0], self.spec.hidden), torch.float32)
         kernels.moe_combine(y, weights, gate, shared, out)
         return out

@@ -37,6 +37,8 @@ def random_tensors(expected: dict, seed: int, std: float = 0.02, gain_spread: fl
             out[name] = t.to(dtype)
         elif getattr(exp, "init", "normal") != "normal":
             raise ValueError(f"tensor {name!r}: unknown random initialisation {exp.init!r}")
+        elif not shape:
+            out[name] = (torch.randn((), generator=g) * std).to(dtype)
         else:
             t = torch.empty(shape, dtype=dtype)
             rows = shape[0]
