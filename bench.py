@@ -466,6 +466,30 @@ def _gavatar_configs(size):
 GAVATAR_WINDOW, GAVATAR_RANK = 1024, 192
 
 
+def _nurilorn_configs(size):
+    """A Nurilorn model of the size's width (four layers of causal attention over convolved projections, capped scores,
+    values mixed with the first layer's; a dense clamped feed-forward, then three layers of 16 experts in four groups of
+    which a token runs four from two groups: as many ACTIVE feed-forward parameters as the dense models) and the Kipezen
+    model of equal width, depth and head geometry, the closest family the engine had (a routed mixture of experts in
+    groups, short convolutions with state, rotated attention with float32 scores)."""
+    from inf_engine_b200.config import parse_config_dict
+    z = FAMILY_SIZES[size]
+    w, H, G, inter = z["width"], z["heads"], z["kv"], z["inter"]
+    att = {"heads": H, "kv_heads": G, "dim": FAMILY_HD, "vdim": FAMILY_HD, "conv": 4, "scale": FAMILY_HD ** -0.5,
+           "softcap": NURILORN_CAP, "v_mix": True,
+           "rot": {"base": 10000.0, "dims": FAMILY_HD // 2, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    dense = {"kind": "dense", "ff": inter, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": inter // 4, "limit": 7.0},
+           "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    layers = [{"type": "attention", "mixer": att, "mlp": dense if i == 0 else moe} for i in range(FAMILY_LAYERS)]
+    nur = parse_config_dict({"architecture": "Nurilorn", "vocab": FAMILY_VOCAB, "width": w, "norm": {"eps": 1e-5, "groups": 4},
+                             "embedding": {"scale": float(w) ** 0.5}, "residual_mult": 0.5, "logit_scale": 0.5, "layers": layers})
+    return nur, _kipezen_configs(size)[0]
+
+
+NURILORN_CAP = 30.0
+
+
 def _weight_bytes(runner):
     seen, n = set(), 0
     import torch
@@ -491,8 +515,8 @@ def run_family(args):
     from inf_engine_b200 import Engine, StepEntry, SamplingConfig, kernels
     from inf_engine_b200.sampling import pack_rows, request_key
 
-    if args.family not in ("barerax", "kipezen", "fovunex", "gavatar"):
-        print(f"--family {args.family}: unknown (known: barerax, kipezen, fovunex, gavatar)")
+    if args.family not in ("barerax", "kipezen", "fovunex", "gavatar", "nurilorn"):
+        print(f"--family {args.family}: unknown (known: barerax, kipezen, fovunex, gavatar, nurilorn)")
         return 2
     pk = peaks()
     torch.cuda.set_device(0)
@@ -1218,8 +1242,161 @@ def run_family(args):
             N * (E * 4 + 4 * 8), N * (E * 4 + 2 * 8 + 4))
         return rows
 
+    def nurilorn_kernel_table(size):
+        """Every kernel that the Nurilorn family added or extended, alone, beside the like kernel of the closest family
+        (Kipezen), at 2,048 tokens of one request and at 8 requests of one token over 2,048 keys."""
+        from inf_engine_b200.engine.batch import KVGroupContext, StepContext
+        from inf_engine_b200.parts import CacheView, Runtime
+        from inf_engine_b200.parts.attention import PagedAttention
+        from inf_engine_b200.parts.latent import attend_float32
+        z = FAMILY_SIZES[size]
+        W, H, G, hd, inter = z["width"], z["heads"], z["kv"], FAMILY_HD, z["inter"]
+        N, B, dev, bf = PROMPT_LEN, 8, "cuda", torch.bfloat16
+        g = torch.Generator(device=dev).manual_seed(1)
+        rnd = lambda *shape: (torch.randn(*shape, device=dev, generator=g) * 0.5)
+        i32 = lambda v: torch.as_tensor(v, dtype=torch.int32, device=dev)
+        rows = []
+
+        def add(name, like, ms, ms_like, nbytes=None, nbytes_like=None, flops=None, flops_like=None, note=None):
+            rec = {"kernel": name, "like": like, "ms": ms, "like_ms": ms_like}
+            if nbytes is not None:
+                rec["frac_of_hbm"] = nbytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"]
+                if ms_like:
+                    rec["like_frac_of_hbm"] = (nbytes_like or nbytes) / (ms_like * 1e-3) / 1e9 / pk["hbm_gbs"]
+            if flops is not None:
+                rec["frac_of_bf16"] = flops / (ms * 1e-3) / 1e12 / pk["bf16_tflops"]
+                if ms_like:
+                    rec["like_frac_of_bf16"] = (flops_like or flops) / (ms_like * 1e-3) / 1e12 / pk["bf16_tflops"]
+            if note:
+                rec["note"] = note
+            rows.append(rec)
+
+        rt = Runtime(dev, bf)
+        n_pages = B * N // PAGE
+        qs1, sl1 = i32([0, N]), i32([0])
+        qs8, sl8 = torch.arange(B + 1, dtype=torch.int32, device=dev), torch.arange(B, dtype=torch.int32, device=dev)
+
+        def context(q_lens, before):
+            ctx = StepContext(rt, PAGE)
+            R, n = len(q_lens), sum(q_lens)
+            ctx.n_tokens, ctx.n_requests, ctx.n_logits = n, R, 0
+            starts = [0]
+            for ql in q_lens:
+                starts.append(starts[-1] + ql)
+            per = n_pages // R
+            ctx.q_start, ctx.ctx_before = i32(starts), i32(before)
+            ctx.positions = i32([b + t for ql, b in zip(q_lens, before) for t in range(ql)])
+            ctx.slots = i32(list(range(R)))
+            table_ = torch.arange(per * R, dtype=torch.int32, device=dev).view(R, per)
+            sm = i32([(r * per + (b + t) // PAGE) * PAGE + (b + t) % PAGE for r, (ql, b) in enumerate(zip(q_lens, before)) for t in range(ql)])
+            ctx.kv = [KVGroupContext(sm, table_)]
+            ctx.host = {"q_lens": list(q_lens), "ctx_before": list(before), "q_start": starts}
+            ctx.max_q_len, ctx.max_seq_len = max(q_lens), max(b + ql for ql, b in zip(q_lens, before))
+            ctx.keys_cap = ctx.max_seq_len
+            return ctx
+
+        ctx_p, ctx_d = context([N], [0]), context([1] * B, [N - 1] * B)
+        pairs_all = N * (N + 1) // 2
+        # the stream
+        ids_v, table_v, res = torch.randint(0, FAMILY_VOCAB, (N,), device=dev, generator=g, dtype=torch.int32), rnd(FAMILY_VOCAB, W).to(bf), rnd(N, W)
+        add("embedding with a multiplier", "embedding",
+            timed(lambda: kernels.embed_gather(ids_v, table_v, res, 3.0)), timed(lambda: kernels.embed_gather(ids_v, table_v, res)),
+            N * W * 6, N * W * 6)
+        E, top, ffe = 16, 4, inter // 4
+        y, yp, wts = rnd(N, W).to(bf), rnd(N * top, W), torch.rand(N, top, device=dev, generator=g)
+        out, gain, gain_b, ls = torch.empty(N, W, device=dev, dtype=bf), 1 + 0.1 * rnd(W), (1 + 0.1 * rnd(W)).to(bf), rnd(W)
+        comb, nxt = torch.empty(N, W, device=dev), torch.empty(N, W, device=dev, dtype=bf)
+        for n, what in ((N, "prompt"), (B, "decode b8")):
+            add(f"scaled sum into the stream + grouped norm (bfloat16 summand), {what}", "norm of a sublayer's output into the residual + next input",
+                timed(lambda: kernels.stream_norm(res[:n], y[:n], ls, None, gain_b, 4, 1e-5, out[:n])),
+                timed(lambda: kernels.outnorm_accumulate(res[:n], y[:n], gain, 1e-5, nxt[:n])), n * W * (4 + 4 + 2 + 2), n * W * (4 + 4 + 2 + 2))
+
+            def like_combine():
+                kernels.moe_combine(yp[:n * top], wts[:n], None, None, comb[:n])
+                kernels.outnorm_accumulate(res[:n], comb[:n], gain, 1e-5, nxt[:n])
+            add(f"experts' weighted sum + scaled sum into the stream + grouped norm, {what}", "experts' weighted sum, norm of it into the residual (two kernels)",
+                timed(lambda: kernels.stream_norm(res[:n], yp[:n * top], ls, wts[:n], gain_b, 4, 1e-5, out[:n])), timed(like_combine),
+                n * W * (4 * top + 4 + 4 + 2), n * W * (4 * top + 4 + 4 + 4 + 4 + 2))
+        # projections to attention operands
+        C = (H + 2 * G) * hd
+        qkv, wt, wb = rnd(N, C + 8).to(bf)[:, :C], rnd(4, C), rnd(C, 4).to(bf)
+        state = torch.zeros(16, 3, C, device=dev, dtype=bf)
+        q = torch.empty(N, H * hd, device=dev, dtype=bf)
+        kpool, vpool = (torch.zeros(n_pages, G, PAGE, hd, device=dev, dtype=bf) for _ in range(2))
+        kept, conv = rnd(N, G * hd).to(bf), torch.empty(N, C, device=dev, dtype=bf)
+        inv_freq = (10000.0 ** (-2.0 * torch.arange(hd // 4, dtype=torch.float64) / (hd // 2))).to(dev)
+        qg, kg = (1 + 0.1 * rnd(H * hd)).to(bf), (1 + 0.1 * rnd(G * hd)).to(bf)
+        for n, ctx, qs, sl, R, what in ((N, ctx_p, qs1, sl1, 1, "prompt"), (B, ctx_d, qs8, sl8, B, "decode b8")):
+            slots_ = ctx.kv[0].slot_mapping
+
+            def like_conv():
+                kernels.causal_conv(qkv[:n], wb, None, state, conv[:n], qs, sl, R, activation="silu", max_q_len=ctx.max_q_len)
+                kernels.rownorm_rotate_write(conv[:n, :H * hd], conv[:n, H * hd:(H + G) * hd], conv[:n, (H + G) * hd:], None, None, None, qg, kg, 1e-5,
+                                             inv_freq, hd // 2, ctx.positions, slots_, kpool, vpool, H, G, hd, hd, PAGE)
+            add(f"convolution + rotation + value mixing + cache write, {what}", "convolution, then norm + rotation + cache write (two kernels)",
+                timed(lambda: kernels.conv_qkv(qkv[:n], wt, state, q[:n], kpool, vpool, ctx.positions, slots_, qs, sl, R, H, G, hd, hd, H * hd,
+                                               (H + G) * hd, PAGE, inv_freq=inv_freq, rot_dims=hd // 2, v_kept=kept[:n], v_mode="mix", lam=0.4,
+                                               max_q_len=ctx.max_q_len)), timed(like_conv),
+                n * (2 * C + G * hd) * 2 + (R * 6 * C * 2 if n == B else 0), n * 4 * C * 2 + (R * 6 * C * 2 if n == B else 0))
+        # attention
+        kpool.normal_(generator=g)
+        vpool.normal_(generator=g)
+        q.normal_(generator=g)
+        spec_k = _kipezen_configs(size)[0].model_spec().layers[3].mixer.branches[0]
+        tensors = {n: ((1 + 0.1 * rnd(*e.shape)) if e.init == "gain" else rnd(*e.shape) * 0.1).to(bf)
+                   for n, e in PagedAttention.expected_tensors(spec_k).items()}
+        att_k = PagedAttention(spec_k, tensors, rt)
+        view_k = CacheView("kv", 0, kpool, vpool, None, True)
+        out_k, out_n = torch.empty(N, H * hd, device=dev, dtype=bf), torch.empty(N, H * hd, device=dev, dtype=bf)
+        like_att = lambda ctx, n: att_k._attend(q[:n], out_k[:n], view_k, ctx, ctx.kv[0], head_scale=att_k.head_scale)
+        window = 1024
+        pairs_k = pairs_all - (N - window) * (N - window + 1) // 2 + 4 * (N - window - 4)
+        sink, gate_ = torch.zeros(H, device=dev), rnd(N, H).to(bf)
+        att = lambda ctx, n, cap=NURILORN_CAP: attend_float32(q[:n], out_n[:n], kpool, vpool, ctx, ctx.kv[0], H, G, hd, hd, 0.125, None,
+                                                              sink=sink, softcap=cap, gate=gate_[:n])
+        like_p, like_d = timed(lambda: like_att(ctx_p, N), reps=5), timed(lambda: like_att(ctx_d, B))
+        add("attention with capped scores, prompt (%d heads over %d)" % (H, G), "attention, prompt (window of 1,024 + 4 kept keys)",
+            timed(lambda: att(ctx_p, N), reps=5), like_p, flops=4 * H * hd * pairs_all, flops_like=4 * H * hd * pairs_k)
+        add("the same without the cap", "attention, prompt (window of 1,024 + 4 kept keys)",
+            timed(lambda: att(ctx_p, N, 0.0), reps=5), like_p, flops=4 * H * hd * pairs_all, flops_like=4 * H * hd * pairs_k)
+        add("attention with capped scores, decode b8 x 2,048 keys (%d heads over %d)" % (H, G), "attention, decode (1,028 visible)",
+            timed(lambda: att(ctx_d, B)), like_d, B * N * G * hd * 2 * 2, B * (window + 4) * G * hd * 2 * 2)
+        # as many key heads as query heads: nothing is shared, decode tokens take the rows kernel
+        kp1, vp1 = (torch.randn(n_pages, H, PAGE, hd, device=dev, generator=g).to(bf) for _ in range(2))
+        att1 = lambda ctx, n: attend_float32(q[:n], out_n[:n], kp1, vp1, ctx, ctx.kv[0], H, H, hd, hd, 0.125, None, sink=sink,
+                                             softcap=NURILORN_CAP, gate=gate_[:n])
+        add("attention with capped scores, prompt (%d heads over %d)" % (H, H), "attention, prompt (window of 1,024 + 4 kept keys)",
+            timed(lambda: att1(ctx_p, N), reps=5), like_p, flops=4 * H * hd * pairs_all, flops_like=4 * H * hd * pairs_k)
+        add("attention with capped scores, decode b8 x 2,048 keys (%d heads over %d)" % (H, H), "attention, decode (1,028 visible)",
+            timed(lambda: att1(ctx_d, B)), like_d, B * N * H * hd * 2 * 2, B * (window + 4) * G * hd * 2 * 2)
+        # feed-forward
+        x = rnd(N, W).to(bf)
+        logits = rnd(N, E + 1) * 2
+        ids4 = torch.empty(N, top, dtype=torch.int32, device=dev)
+        w4, gt = torch.empty(N, top, device=dev), torch.empty(N, device=dev)
+        add("router: softmax scores, 4 of 16 from 2 of 4 groups", "router: sigmoid scores, 4 of 16 from 2 of 4 groups",
+            timed(lambda: kernels.moe_route(logits[:, :E], None, ids4, w4, None, E, top, 4, 2, 1.0, 1e-20, score="softmax", group_score="max")),
+            timed(lambda: kernels.moe_route(logits, None, ids4, w4, gt, E, top, 4, 2, 2.5, 1e-20, gate_col=E)),
+            N * (E * 4 + top * 8), N * (E * 4 + top * 8 + 4))
+        kernels.moe_route(logits[:, :E], None, ids4, w4, None, E, top, 4, 2, 1.0, 1e-20, score="softmax", group_score="max")
+        gate_up, act = (rnd(E, 2 * ffe, W) * 0.1).to(bf), (1.702, 7.0, 1.0)
+        hid = torch.empty(N * top, ffe, device=dev, dtype=bf)
+        for n, what in ((N, "prompt"), (B, "decode b8")):
+            pairs_ = torch.empty(n * top, dtype=torch.int32, device=dev)
+            tiles = torch.empty(kernels.moe_max_tiles(n * top, E), 4, dtype=torch.int32, device=dev)
+            kernels.moe_sort(ids4[:n], E, pairs_, tiles)
+            run = lambda a: kernels.moe_gemm(x[:n], gate_up, hid[:n * top], pairs_, tiles, top, gather=True, scatter=False, epi="silu_mul", act=a)
+            chosen = len(set(ids4[:n].flatten().tolist()))
+            kw = dict(flops=2 * n * top * 2 * ffe * W) if n == N else dict(nbytes=chosen * 2 * ffe * W * 2)
+            add(f"experts' gate/up product with the clamped activation, {what}", "the same with SiLU", timed(lambda: run(act)), timed(lambda: run(None)), **kw)
+        dense_w, dense_out = (rnd(2 * inter, W) * 0.1).to(bf), torch.empty(N, inter, device=dev, dtype=bf)
+        add("dense gate/up product with the clamped activation, prompt", "the same with SiLU",
+            timed(lambda: kernels.gemm_tcgen05(x, dense_w, dense_out, "silu_mul", act=act)),
+            timed(lambda: kernels.gemm_tcgen05(x, dense_w, dense_out, "silu_mul")), flops=2 * N * 2 * inter * W)
+        return rows
+
     sizes = {}
-    if args.family in ("kipezen", "fovunex", "gavatar") and args.family_step:
+    if args.family in ("kipezen", "fovunex", "gavatar", "nurilorn") and args.family_step:
         # one step launched kernel by kernel (no graphs) between cudaProfilerStart / Stop, for a launch list:
         #   ncu --metrics gpu__time_duration.sum --clock-control none --profile-from-start off --csv --log-file L \
         #       python bench.py --family kipezen --family-sizes w2048 --family-step decode
@@ -1227,7 +1404,8 @@ def run_family(args):
         from inf_engine_b200 import ModelRunner
         from inf_engine_b200.weights import write_random_model
         size = (args.family_sizes or "w2048").split(",")[0]
-        kpz, _ = {"kipezen": _kipezen_configs, "fovunex": _fovunex_configs, "gavatar": _gavatar_configs}[args.family](size)
+        kpz, _ = {"kipezen": _kipezen_configs, "fovunex": _fovunex_configs, "gavatar": _gavatar_configs,
+                  "nurilorn": _nurilorn_configs}[args.family](size)
         with tempfile.TemporaryDirectory() as tmp:
             write_random_model(kpz, args.seed, tmp)
             r = ModelRunner.from_dir(tmp, dtype="bfloat16", page_size=PAGE, n_pages=(args.batch + 1) * POOL_CONTEXT // PAGE,
@@ -1254,6 +1432,23 @@ def run_family(args):
         torch.cuda.cudart().cudaProfilerStop()
         clocks.stop()
         print(json.dumps({"impl": "ours", "family": args.family, "step": args.family_step, "size": size, "launches": kernels.LAUNCHES}))
+        return 0
+    if args.family == "nurilorn":
+        for size in (args.family_sizes.split(",") if args.family_sizes else list(FAMILY_SIZES)):
+            nur, kpz = _nurilorn_configs(size)
+            rec = {"nurilorn": model_numbers_of(nur, args.batch), "kipezen": model_numbers_of(kpz, args.batch)}
+            rec["kernels"] = nurilorn_kernel_table(size)
+            sizes[size] = rec
+        clocks.stop()
+        print(json.dumps({"impl": "ours", "family": "nurilorn", "dtype": "bf16", "n_gpus": 1, "steps": args.steps,
+                          "warmup": max(args.warmup, 3),
+                          "data": "synthetic: seeded random weights, uniform random prompt ids",
+                          "config": {"layers": FAMILY_LAYERS, "pattern": "attention with a dense feed-forward, then three with experts",
+                                     "vocab": FAMILY_VOCAB, "head_dim": FAMILY_HD, "prompt": PROMPT_LEN, "decode_batch": args.batch,
+                                     "page_size": PAGE, "taps": 4, "softcap": NURILORN_CAP, "experts": "16 in 4 groups, 4 a token from 2 groups",
+                                     "l2": "a 256 MB buffer is written before every timed kernel; model steps stream their weights",
+                                     "sizes": FAMILY_SIZES},
+                          "peaks": pk, "sizes": sizes, "clocks": clocks.summary(t_all0, time.perf_counter())}))
         return 0
     if args.family == "gavatar":
         for size in (args.family_sizes.split(",") if args.family_sizes else list(FAMILY_SIZES)):
@@ -1508,11 +1703,11 @@ def main():
     ap.add_argument("--no-workloads", action="store_true",
                     help="leave out the two continuous-batching workloads at the other models' sizes")
     ap.add_argument("--family", default=None, metavar="NAME",
-                    help="instead of the default workload: prefill and decode of another model family (barerax, kipezen, fovunex, gavatar) at sizes like "
+                    help="instead of the default workload: prefill and decode of another model family (barerax, kipezen, fovunex, gavatar, nurilorn) at sizes like "
                          "a real model's layers, beside the closest earlier model of equal size, and its kernels beside the like ones")
     ap.add_argument("--family-sizes", default=None, help="comma-separated subset of the family's sizes (w1024,w2048)")
     ap.add_argument("--family-step", default=None, choices=["decode", "prefill"],
-                    help="with --family kipezen, fovunex or gavatar: run one such step kernel by kernel between cudaProfilerStart/Stop (for a launch list) and exit")
+                    help="with --family kipezen, fovunex, gavatar or nurilorn: run one such step kernel by kernel between cudaProfilerStart/Stop (for a launch list) and exit")
     ap.add_argument("--workload", default=None, metavar="N:MIN:MAX:NEW[:TEMP]",
                     help="instead of the step measurements: N requests through Engine.run_offline (continuous batching)")
     args = ap.parse_args()
