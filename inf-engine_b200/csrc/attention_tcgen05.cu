@@ -24,6 +24,13 @@
 //               about as long as the softmax of a tile takes: with one issuing thread for both products the
 //               softmax waited for it half of the time
 //
+// Built with -DIE_FA_EXACT=1 the same kernel keeps the softmax weights in 32 bits: a weight meets the values as two
+// bfloat16 terms (its rounding and what that left out), which share the columns of the S buffer it was made from, and
+// the denominator may hold one more term exp(sink[head]), the output a sigmoid gate of one number a head.  With capped
+// scores (softcap * tanh(s / softcap)) no score exceeds the cap, so the exponentials are taken relative to a fixed 0:
+// there is no maximum to find and O is never rescaled (caps up to 60: e^60 times any number of keys stays far inside
+// float32, and a denominator of e^-60 too).
+//
 // Every wait on an mbarrier is bounded; on a timeout the block records an error word, stops, frees its tensor
 // memory and leaves.
 #include "common.cuh"
@@ -82,7 +89,16 @@ struct FaParams {
   const float* cos_t;
   const float* sin_t;
   const int* positions;
+  // the exact build (MODE > 0)
+  const float* sink;       // [n_heads] or null
+  const bf16* gate;        // [tokens, n_heads] or null
+  int gate_stride;
+  float cap_in, cap_log2;  // scale / softcap and softcap log2 e (MODE 2)
 };
+
+// MODE 0: weights are rounded to bfloat16.  MODE 1: weights in two bfloat16 terms, a running maximum, a sink, a gate.
+// MODE 2: the same with capped scores and no maximum.
+[[maybe_unused]] constexpr float FA_MAX_CAP = 60.f;
 
 __device__ __forceinline__ uint32_t saddr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void fa_mbar_init(uint32_t bar, int count) {
@@ -181,6 +197,11 @@ __device__ __forceinline__ void fa_tmem_st16(uint32_t taddr, const uint32_t (&r)
         "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
       : "memory");
 }
+__device__ __forceinline__ void fa_tmem_st8(uint32_t taddr, const uint32_t* r) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};"
+               ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7])
+               : "memory");
+}
 __device__ __forceinline__ float fa_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
@@ -204,9 +225,19 @@ __device__ __forceinline__ uint64_t fa_add2(uint64_t a, uint64_t b) {
   asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
+__device__ __forceinline__ uint64_t fa_mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 __device__ __forceinline__ float fa_max3(float a, float b, float c) {
   float d;
   asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+[[maybe_unused]] __device__ __forceinline__ float fa_min3(float a, float b, float c) {
+  float d;
+  asm("min.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
   return d;
 }
 __device__ __forceinline__ uint32_t fa_pack(float lo, float hi) {
@@ -216,7 +247,7 @@ __device__ __forceinline__ uint32_t fa_pack(float lo, float hi) {
 // byte offset of 16-byte chunk `chunk` (0..7) of row `row` in a tile of 128-byte rows under the 128-byte swizzle
 __device__ __forceinline__ uint32_t sw128(int row, int chunk) { return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4)); }
 
-template <int HD, int KT, int STAGES, int PBUF, int SBUF>
+template <int HD, int KT, int STAGES, int PBUF, int SBUF, int MODE>
 __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::BLOCKS_PER_SM) attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                                                                           const __grid_constant__ CUtensorMap map_v,
                                                                           FaParams p) {
@@ -224,6 +255,7 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
   // p_ready[2], pv_done[2], q_ready), the tensor-memory slot and the failure flag.  No static shared memory and no
   // padding: two blocks have to fit one SM.
   using G = Geo<HD, KT, STAGES, PBUF, SBUF>;
+  static_assert(MODE == 0 || PBUF == 0, "two terms of a weight take the S buffer's own columns");
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned long long* bars = reinterpret_cast<unsigned long long*>(smem_raw + G::TILES_BYTES);
   uint32_t* tmem_slot_p = reinterpret_cast<uint32_t*>(smem_raw + G::TILES_BYTES + 120);
@@ -373,6 +405,11 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
 #pragma unroll
           for (int kk = 0; kk < KT / 16; ++kk)
             fa_umma_ts(tmem_o, pa + (uint32_t)(kk * 8), vd + (uint64_t)((kk * 2048) >> 4), idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+          if constexpr (MODE > 0) {        // what the first term left out: the other KT/2 columns
+#pragma unroll
+            for (int kk = 0; kk < KT / 16; ++kk)
+              fa_umma_ts(tmem_o, pa + (uint32_t)(KT / 2 + kk * 8), vd + (uint64_t)((kk * 2048) >> 4), idesc_o, 1u);
+          }
         }
         // K of the stage was read by S_j, which was complete before the softmax of tile j read it; V by these
         fa_commit(kv_empty0 + 8 * s);
@@ -449,7 +486,7 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
       return true;
     };
 
-    float m = -INFINITY, l = 0.f;
+    float m = MODE == 2 ? 0.f : -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       ok = wait_all(s_full0 + 8 * (j & 1), (uint32_t)(j >> 1) & 1u, 4);
@@ -460,7 +497,7 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
       // the scores of the row are read twice from tensor memory (once for the maximum, once for the exponentials),
       // each time with all loads on their way before the one wait
       float mx = -INFINITY;
-      {
+      if constexpr (MODE != 2) {
         float sc[KT];
 #pragma unroll
         for (int q4 = 0; q4 < KT / 32; ++q4) fa_tmem_ld32_issue(tmem_s + lane_addr + (j % SBUF) * KT + q4 * 32, sc + q4 * 32);
@@ -483,8 +520,8 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
       // first): until then the exponentials are at most 256, which neither bfloat16 nor the float32 sums
       // mind, and O in tensor memory needs no rescaling.  The result is the same: numerator and
       // denominator carry the same factor.
-      const float m_cand = fmaxf(m, mx * p.scale_log2);
-      const bool moves = __any_sync(0xffffffffu, m_cand - m > 8.f || (m == -INFINITY && m_cand > -INFINITY));
+      const float m_cand = MODE == 2 ? 0.f : fmaxf(m, mx * p.scale_log2);
+      const bool moves = MODE != 2 && __any_sync(0xffffffffu, m_cand - m > 8.f || (m == -INFINITY && m_cand > -INFINITY));
       float corr = 1.f;
       if (moves) {
         corr = fa_exp2(m - (m_cand == -INFINITY ? 0.f : m_cand));    // 2^(-inf) = 0 the first time
@@ -520,17 +557,50 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
       auto exp_pass = [&](auto masked) {
         constexpr bool MASKED = decltype(masked)::value;
         uint32_t pk[16];
+        [[maybe_unused]] uint32_t pl[8];
         float sc[KT];
 #pragma unroll
         for (int q4 = 0; q4 < KT / 32; ++q4) fa_tmem_ld32_issue(tmem_s + lane_addr + (j % SBUF) * KT + q4 * 32, sc + q4 * 32);
         fa_tmem_wait_ld();
+        if constexpr (MODE == 2) {
+          // capped scores in the exponent's units, in place.  Where every score of the warp's tile lies well below the
+          // cap the hyperbolic tangent is a polynomial (no trip to the special-function unit); else 1 - 2 / (1 + e^2z).
+          float hi = 0.f, lo = 0.f;
+#pragma unroll
+          for (int i = 0; i < KT; i += 2) {
+            hi = fa_max3(hi, sc[i], sc[i + 1]);
+            lo = fa_min3(lo, sc[i], sc[i + 1]);
+          }
+          if (__all_sync(0xffffffffu, fmaxf(hi, -lo) * p.cap_in <= TANH_SMALL)) {
+            const float coef[5] = {TANH_COEFS};
+            const uint64_t c2 = fa_pair(p.cap_in, p.cap_in);
+            uint64_t a[5];
+#pragma unroll
+            for (int k = 0; k < 5; ++k) a[k] = fa_pair(coef[k] * p.cap_log2, coef[k] * p.cap_log2);
+#pragma unroll
+            for (int i = 0; i < KT; i += 2) {
+              const uint64_t zz = fa_mul2(fa_pair(sc[i], sc[i + 1]), c2), u = fa_mul2(zz, zz);
+              const uint64_t q01 = fa_fma2(u, fa_fma2(u, fa_fma2(u, fa_fma2(u, a[4], a[3]), a[2]), a[1]), a[0]);
+              fa_unpair(fa_mul2(zz, q01), sc[i], sc[i + 1]);
+            }
+          } else {
+            const float c1 = 2.f * LOG2E * p.cap_in, down = -2.f * p.cap_log2;
+#pragma unroll
+            for (int i = 0; i < KT; ++i) sc[i] = fmaf(down, __fdividef(1.f, 1.f + fa_exp2(sc[i] * c1)), p.cap_log2);
+          }
+        }
 #pragma unroll
         for (int ch = 0; ch < KT / 8; ++ch) {
           float e[8];
 #pragma unroll
           for (int i = 0; i < 8; i += 2) {
             float x0, x1;
-            fa_unpair(fa_fma2(fa_pair(sc[ch * 8 + i], sc[ch * 8 + i + 1]), scale2, neg_m2), x0, x1);
+            if constexpr (MODE == 2) {
+              x0 = sc[ch * 8 + i];
+              x1 = sc[ch * 8 + i + 1];
+            } else {
+              fa_unpair(fa_fma2(fa_pair(sc[ch * 8 + i], sc[ch * 8 + i + 1]), scale2, neg_m2), x0, x1);
+            }
             x0 = fa_exp2(x0);
             x1 = fa_exp2(x1);
             e[i] = (!MASKED || k0 + ch * 8 + i <= limit) ? x0 : 0.f;
@@ -543,9 +613,23 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
           if (PBUF > 0) {
             *reinterpret_cast<uint4*>(p_tile + (col >> 6) * ATOM_BYTES + sw128(r, (col & 63) >> 3)) = v;
           } else {
-            // 32 keys (16 columns) at a time into the S buffer's own columns: every score of the tile is in registers
-            pk[(ch & 3) * 4] = v.x; pk[(ch & 3) * 4 + 1] = v.y; pk[(ch & 3) * 4 + 2] = v.z; pk[(ch & 3) * 4 + 3] = v.w;
-            if ((ch & 3) == 3) fa_tmem_st16(p_tmem + (uint32_t)((ch >> 2) * 16), pk);
+            // 32 keys (16 columns; in two terms 16 keys, 8 columns of each) at a time into the S buffer's own columns:
+            // every score of the tile is in registers
+            constexpr int W = MODE > 0 ? 2 : 4;
+            pk[(ch % W) * 4] = v.x; pk[(ch % W) * 4 + 1] = v.y; pk[(ch % W) * 4 + 2] = v.z; pk[(ch % W) * 4 + 3] = v.w;
+            if constexpr (MODE == 0) {
+              if (ch % W == W - 1) fa_tmem_st16(p_tmem + (uint32_t)((ch / W) * 16), pk);
+            } else {
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pk[(ch % W) * 4 + i]));
+                pl[(ch % W) * 4 + i] = fa_pack(e[2 * i] - h.x, e[2 * i + 1] - h.y);
+              }
+              if (ch % W == W - 1) {
+                fa_tmem_st8(p_tmem + (uint32_t)((ch / W) * 8), pk);
+                fa_tmem_st8(p_tmem + (uint32_t)(KT / 2 + (ch / W) * 8), pl);
+              }
+            }
           }
         }
       };
@@ -588,7 +672,17 @@ __global__ void __launch_bounds__(FA_THREADS, Geo<HD, KT, STAGES, PBUF, SBUF>::B
     }
     if (ok) ok = wait_all(pv_done0 + 8 * ((n_tiles - 1) & 1), (uint32_t)((n_tiles - 1) >> 1) & 1u, 7);
     if (ok) {
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if constexpr (MODE > 0) {
+        if (p.sink != nullptr && valid && m > -INFINITY) {
+          // the sink's term joins at the larger of the two references
+          const float sk = p.sink[head] * LOG2E, m2 = fmaxf(m, sk);
+          const float f = exp2f(m - m2);
+          inv = f / (l * f + exp2f(sk - m2));
+        }
+        if (p.gate != nullptr && valid)
+          inv *= 1.f / (1.f + expf(-to_f32(p.gate[(size_t)(q0 + t) * p.gate_stride + head])));
+      }
       bf16* dst = p.out + (size_t)(q0 + t) * p.out_stride + head * HD;
 #pragma unroll
       for (int h = 0; h < HD / 32; ++h) {
@@ -667,20 +761,45 @@ extern "C" int ie_attention_tcgen05_supports(int hd, int page_size, int window) 
   return 1;
 }
 
-template <int HD, int KT, int STAGES, int PBUF, int SBUF>
+template <int HD, int KT, int STAGES, int PBUF, int SBUF, int MODE = 0>
 static int fa_launch(const CUtensorMap& mk, const CUtensorMap& mv, const FaParams& p, int n_work, int n_kv_heads,
                      cudaStream_t stream) {
   const size_t smem = Geo<HD, KT, STAGES, PBUF, SBUF>::TILES_BYTES + 128;
   static bool attr = false;
   if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<HD, KT, STAGES, PBUF, SBUF>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<HD, KT, STAGES, PBUF, SBUF, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     attr = true;
   }
-  return launch_k(attention_tcgen05_kernel<HD, KT, STAGES, PBUF, SBUF>, dim3((unsigned)((long long)n_work * n_kv_heads)), FA_THREADS, smem,
+  return launch_k(attention_tcgen05_kernel<HD, KT, STAGES, PBUF, SBUF, MODE>, dim3((unsigned)((long long)n_work * n_kv_heads)), FA_THREADS, smem,
                   stream, mk, mv, p);
 }
 
+static int fa_setup(CUtensorMap& mk, CUtensorMap& mv, FaParams& p, const void* q, void* out, const void* kpool, const void* vpool,
+                    const int* block_table, const int* q_start, const int* ctx_before, const int* work_req,
+                    const int* work_pair0, int q_stride, int out_stride, int table_stride, int n_work, int n_heads,
+                    int n_kv_heads, int hd, int page_size, int n_pool_pages, float scale) {
+  if (!ie_attention_tcgen05_supports(hd, page_size, 0)) return IE_BAD_SIZE;
+  if (n_kv_heads <= 0 || n_heads % n_kv_heads || n_pool_pages <= 0) return IE_BAD_SIZE;
+  if (((uintptr_t)q | (uintptr_t)out | (uintptr_t)kpool | (uintptr_t)vpool) & 15) return IE_BAD_ALIGN;
+  if ((q_stride | out_stride) & 7) return IE_BAD_ALIGN;
+  const long long rows = (long long)n_pool_pages * n_kv_heads * page_size;
+  int rc = fa_make_map(&mk, kpool, rows, page_size, hd);
+  if (rc) return rc;
+  rc = fa_make_map(&mv, vpool, rows, page_size, hd);
+  if (rc) return rc;
+  p = FaParams{};
+  p.q = (const bf16*)q; p.out = (bf16*)out; p.block_table = block_table; p.q_start = q_start; p.ctx_before = ctx_before;
+  p.work_req = work_req; p.work_pair0 = work_pair0; p.q_stride = q_stride; p.out_stride = out_stride;
+  p.table_stride = table_stride; p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.page_size = page_size;
+  p.n_work = n_work;
+  p.page_shift = 0;
+  while ((1 << p.page_shift) < page_size) ++p.page_shift;
+  p.scale_log2 = scale * LOG2E;
+  return IE_OK;
+}
+
+#if !(defined(IE_FA_EXACT) && IE_FA_EXACT)
 // The work list cuts each request's (token, head-in-group) rows into tiles of 128; n_pool_pages is the
 // number of pages of kpool / vpool; with cos_t / sin_t / positions q arrives unrotated and is rotated as it is read ([pages, kv_heads, page_size, hd]).
 extern "C" int ie_attention_tcgen05(const void* q, void* out, const void* kpool, const void* vpool,
@@ -692,24 +811,11 @@ extern "C" int ie_attention_tcgen05(const void* q, void* out, const void* kpool,
   if (n_work <= 0) return IE_OK;
   if ((cos_t == nullptr) != (sin_t == nullptr) || (cos_t && !positions)) return IE_BAD_SIZE;
   if (cos_t && (((uintptr_t)cos_t | (uintptr_t)sin_t) & 15)) return IE_BAD_ALIGN;
-  if (!ie_attention_tcgen05_supports(hd, page_size, 0)) return IE_BAD_SIZE;
-  if (n_kv_heads <= 0 || n_heads % n_kv_heads || n_pool_pages <= 0) return IE_BAD_SIZE;
-  if (((uintptr_t)q | (uintptr_t)out | (uintptr_t)kpool | (uintptr_t)vpool) & 15) return IE_BAD_ALIGN;
-  if ((q_stride | out_stride) & 7) return IE_BAD_ALIGN;
   CUtensorMap mk, mv;
-  const long long rows = (long long)n_pool_pages * n_kv_heads * page_size;
-  int rc = fa_make_map(&mk, kpool, rows, page_size, hd);
-  if (rc) return rc;
-  rc = fa_make_map(&mv, vpool, rows, page_size, hd);
-  if (rc) return rc;
   FaParams p;
-  p.q = (const bf16*)q; p.out = (bf16*)out; p.block_table = block_table; p.q_start = q_start; p.ctx_before = ctx_before;
-  p.work_req = work_req; p.work_pair0 = work_pair0; p.q_stride = q_stride; p.out_stride = out_stride;
-  p.table_stride = table_stride; p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.page_size = page_size;
-  p.n_work = n_work;
-  p.page_shift = 0;
-  while ((1 << p.page_shift) < page_size) ++p.page_shift;
-  p.scale_log2 = scale * LOG2E;
+  const int rc = fa_setup(mk, mv, p, q, out, kpool, vpool, block_table, q_start, ctx_before, work_req, work_pair0, q_stride,
+                          out_stride, table_stride, n_work, n_heads, n_kv_heads, hd, page_size, n_pool_pages, scale);
+  if (rc != IE_OK) return rc;
   p.cos_t = cos_t; p.sin_t = sin_t; p.positions = positions;
   // head size 64: two P buffers beside a ring of four stages (two blocks an SM); at 128 the ring takes that room.
   // (-DIE_FA_KT64=128 -DIE_FA_STAGES64=2 -DIE_FA_PBUF64=1 -DIE_FA_SBUF64=1, key tiles of 128 with one S buffer, was
@@ -730,5 +836,36 @@ extern "C" int ie_attention_tcgen05(const void* q, void* out, const void* kpool,
 #endif
   return fa_launch<128, 64, 2, IE_FA_PBUF128, 2>(mk, mv, p, n_work, n_kv_heads, stream);
 }
+
+#else
+
+extern "C" float ie_attention_tcgen05_max_cap() { return FA_MAX_CAP; }
+
+// The exact build: softcap > 0 caps the scores (at most FA_MAX_CAP), `sink` [n_heads] and `gate` [tokens, n_heads] are
+// optional; `scale` must be positive (the running maximum is that of the raw scores).
+extern "C" int ie_attention_tcgen05_exact(const void* q, void* out, const void* kpool, const void* vpool,
+                                          const int* block_table, const int* q_start, const int* ctx_before,
+                                          const int* work_req, const int* work_pair0, int q_stride, int out_stride,
+                                          int table_stride, int n_work, int n_heads, int n_kv_heads, int hd,
+                                          int page_size, int n_pool_pages, float scale, float softcap, const float* sink,
+                                          const void* gate, int gate_stride, cudaStream_t stream) {
+  if (n_work <= 0) return IE_OK;
+  if (!(scale > 0.f) || softcap > FA_MAX_CAP) return IE_BAD_SIZE;
+  CUtensorMap mk, mv;
+  FaParams p;
+  const int rc = fa_setup(mk, mv, p, q, out, kpool, vpool, block_table, q_start, ctx_before, work_req, work_pair0, q_stride,
+                          out_stride, table_stride, n_work, n_heads, n_kv_heads, hd, page_size, n_pool_pages, scale);
+  if (rc != IE_OK) return rc;
+  p.sink = sink; p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
+  if (softcap > 0.f) {
+    p.cap_in = scale / softcap;
+    p.cap_log2 = softcap * LOG2E;
+    if (hd == 64) return fa_launch<64, 64, 4, 0, 2, 2>(mk, mv, p, n_work, n_kv_heads, stream);
+    return fa_launch<128, 64, 2, 0, 2, 2>(mk, mv, p, n_work, n_kv_heads, stream);
+  }
+  if (hd == 64) return fa_launch<64, 64, 4, 0, 2, 1>(mk, mv, p, n_work, n_kv_heads, stream);
+  return fa_launch<128, 64, 2, 0, 2, 1>(mk, mv, p, n_work, n_kv_heads, stream);
+}
+#endif
 
 IE_CHECK_API(attention_tcgen05)

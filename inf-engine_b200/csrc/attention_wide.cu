@@ -53,12 +53,13 @@ struct WideParams {
   int v_row;       // elements between two value rows of the value pool
   int alias;       // the values are the first DV dimensions of the key rows: the key tile is the value tile
   float scale_log2;
-  float cap_in, cap_out;   // the build with capped scores: 2 log2 e scale / softcap, and softcap log2 e
+  float cap_in, cap_out;   // the build with capped scores: scale / softcap, and softcap log2 e
   const bf16* gate;        // [tokens, n_heads] or null: a head's output times sigmoid(gate)
   int gate_stride;
   // without a work list (work_req null): block x is tile x % tiles of request x / tiles, and only requests that bring
   // at most max_rows (token, head-in-group) pairs take part (decode tokens; the others are a work list's)
   int tiles, max_rows;
+  int n_work;
   // n_splits > 1: block z takes the keys [first + z * split_keys, first + (z + 1) * split_keys) of its tile's range
   // (split_keys a multiple of the key tile) and leaves sums, maxima and unnormalised outputs for the merge kernel
   int n_splits, split_keys;
@@ -139,14 +140,17 @@ __device__ __forceinline__ float wide_inv(float l, float m, const float* sink, i
   return f / (l * f + exp2f(sk - m2));
 }
 
-// softcap * tanh(s / softcap) in the exponent's base-2 units, tanh(z) = 1 - 2 / (1 + e^(2 z)): off by a few units of the
-// last place of 1 at most, times softcap, which is the size of the rounding of a score near the cap
-__device__ __forceinline__ float score_log2(float dot, const WideParams& p) {
-#if IE_AW_CAP
-  return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(dot * p.cap_in)));
-#else
-  return dot * p.scale_log2;
-#endif
+// softcap * tanh(s / softcap) in the exponent's base-2 units.  `small`: every score of the warp's tile lies well below the
+// cap, where the hyperbolic tangent is a polynomial; else tanh(z) = 1 - 2 / (1 + e^(2 z)), off by a few units of the last
+// place of 1 at most, times softcap, which is the size of the rounding of a score near the cap.
+[[maybe_unused]] __device__ __forceinline__ float capped_log2(float dot, const WideParams& p, bool small) {
+  const float z = dot * p.cap_in;
+  if (small) {
+    const float a[5] = {TANH_COEFS};
+    const float u = z * z;
+    return p.cap_out * z * fmaf(u, fmaf(u, fmaf(u, fmaf(u, a[4], a[3]), a[2]), a[1]), a[0]);
+  }
+  return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(z * (2.f * LOG2E))));
 }
 
 __device__ __forceinline__ float wide_gate(const WideParams& p, int token, int head) {
@@ -162,9 +166,13 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
   bf16* Kbuf = Qs + BM * LDK;                     // [2][BN][LDK]
   bf16* Vbuf = Kbuf + 2 * BN * LDK;               // [2][BN][LDV] (unused when the values are in the keys)
 
-  const int r_id = p.work_req != nullptr ? p.work_req[blockIdx.x] : (int)blockIdx.x / p.tiles;
-  const int pair0 = p.work_req != nullptr ? p.work_pair0[blockIdx.x] : ((int)blockIdx.x % p.tiles) * BM;
-  const int c = blockIdx.y;
+  // with a work list key heads are the fast index and the list is walked from its end: in a long prompt the tiles with
+  // the most keys start first, and the short ones fill the tail of the launch
+  const bool listed = p.work_req != nullptr;
+  const int w_id = listed ? p.n_work - 1 - (int)blockIdx.x / p.n_kv_heads : 0;
+  const int r_id = listed ? p.work_req[w_id] : (int)blockIdx.x / p.tiles;
+  const int pair0 = listed ? p.work_pair0[w_id] : ((int)blockIdx.x % p.tiles) * BM;
+  const int c = listed ? (int)blockIdx.x % p.n_kv_heads : (int)blockIdx.y;
   const int group = p.n_heads / p.n_kv_heads;
   const int cv = c / (p.n_kv_heads / p.n_v_heads);
   const int q0 = p.q_start[r_id];
@@ -257,6 +265,28 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
 
     // mask, scale, running maximum (exponent units: scale * log2 e is in the multiplier)
     float mx[2] = {-INFINITY, -INFINITY};
+#if IE_AW_CAP
+    {
+      float big = 0.f;
+#pragma unroll
+      for (int nt = 0; nt < NT_S; ++nt)
+        big = fmaxf(big, fmaxf(fmaxf(fabsf(s[nt][0]), fabsf(s[nt][1])), fmaxf(fabsf(s[nt][2]), fabsf(s[nt][3]))));
+      if (__all_sync(0xffffffffu, big * fabsf(p.cap_in) <= TANH_SMALL)) {
+#pragma unroll
+        for (int nt = 0; nt < NT_S; ++nt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[nt][e] = capped_log2(s[nt][e], p, true);
+      } else {
+#pragma unroll
+        for (int nt = 0; nt < NT_S; ++nt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[nt][e] = capped_log2(s[nt][e], p, false);
+      }
+    }
+    constexpr float to_log2 = 1.f;
+#else
+    const float to_log2 = p.scale_log2;
+#endif
 #pragma unroll
     for (int nt = 0; nt < NT_S; ++nt) {
 #pragma unroll
@@ -264,7 +294,7 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
         const int h = e >> 1;
         const int kp = kt + nt * 8 + 2 * t4 + (e & 1);
         const bool vis = kp >= lo[h] && kp <= limit[h];
-        const float v = vis ? score_log2(s[nt][e], p) : -INFINITY;
+        const float v = vis ? s[nt][e] * to_log2 : -INFINITY;
         s[nt][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -439,10 +469,10 @@ static int wide_params(WideParams& p, const void* q, void* out, const void* kpoo
   p.n_v_heads = n_v_heads; p.v_row = v_row; p.sink = sink;
   p.alias = (vpool == kpool && v_row == DK && n_v_heads == n_kv_heads && DV <= DK) ? 1 : 0;
   p.scale_log2 = scale * LOG2E;
-  p.cap_in = softcap > 0.f ? 2.f * LOG2E * scale / softcap : 0.f;
+  p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
   p.cap_out = softcap * LOG2E;
   p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
-  p.tiles = 1; p.max_rows = 0; p.n_splits = 1; p.split_keys = 0; p.part_o = nullptr; p.part_ml = nullptr;
+  p.tiles = 1; p.max_rows = 0; p.n_work = 0; p.n_splits = 1; p.split_keys = 0; p.part_o = nullptr; p.part_ml = nullptr;
   return IE_OK;
 }
 
@@ -463,11 +493,11 @@ extern "C" int ie_attention_wide(const void* q, void* out, const void* kpool, co
                              n_heads, n_kv_heads, page_size, window, scale, chunk, n_v_heads, v_row, sink, softcap, gate,
                              gate_stride);
   if (rc != IE_OK) return rc;
-  p.work_req = work_req; p.work_pair0 = work_pair0;
+  p.work_req = work_req; p.work_pair0 = work_pair0; p.n_work = n_work;
   const size_t smem = wide_smem(p);
   cudaError_t e = cudaFuncSetAttribute(attention_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  return launch_k(attention_wide_kernel, dim3(n_work, n_kv_heads), THREADS, smem, stream, p);
+  return launch_k(attention_wide_kernel, dim3((unsigned)((long long)n_work * n_kv_heads)), THREADS, smem, stream, p);
 }
 
 // floats of scratch that ie_attention_wide_small needs

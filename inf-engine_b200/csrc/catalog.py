@@ -11,6 +11,7 @@ def all_build_requests():
     reqs.append(("stream", ["gemm_stream.cu", "gemm_stream_tma.cu"], {}, []))
     reqs.append(("tcgen05", ["gemm_tcgen05.cu"], {}, []))
     reqs.append(("attn_tcgen05", ["attention_tcgen05.cu"], {}, []))
+    reqs.append(("attn_tcgen05_exact", ["attention_tcgen05.cu"], {"IE_FA_EXACT": 1}, []))
     for hd in (64, 128):
         reqs.append((f"attn_mma_hd{hd}", ["attention_mma.cu"], {"IE_HD": hd}, ["attention_noalloc.h"]))
         reqs.append((f"attn_mma_hd{hd}_bias", ["attention_mma.cu"], {"IE_HD": hd, "IE_ATTN_BIAS": 1}, ["attention_noalloc.h"]))

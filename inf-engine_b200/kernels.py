@@ -1411,6 +1411,65 @@ def attention_tcgen05_library():
     return _fa5_lib
 
 
+_fa5_exact_lib = None
+
+
+def attention_tcgen05_exact_library():
+    """The build of the tcgen05 attention whose softmax weights keep 32 bits; compiled when first asked for."""
+    global _fa5_exact_lib
+    if _fa5_exact_lib is None:
+        lib = load_library("attn_tcgen05_exact", ["attention_tcgen05.cu"],
+                           {"IE_FA_EXACT": 1, **BUILD_DEFINES.get("attn_tcgen05", {})})
+        P, I, F = c_void_p, c_int, c_float
+        lib.ie_attention_tcgen05_exact.argtypes = [P] * 9 + [I] * 9 + [F, F, P, P, I, P]
+        lib.ie_attention_tcgen05_exact.restype = c_int
+        lib.ie_attention_tcgen05_supports.argtypes = [I, I, I]
+        lib.ie_attention_tcgen05_supports.restype = c_int
+        lib.ie_attention_tcgen05_error.restype = c_int
+        lib.ie_attention_tcgen05_max_cap.restype = c_float
+        _fa5_exact_lib = lib
+        _apply_check_limits()
+    return _fa5_exact_lib
+
+
+ATTENTION_TCGEN05_ROWS = 128     # (token, head-in-group) pairs of a tile of the tcgen05 kernels
+
+
+def attention_tcgen05_exact_supports(q, out, kpool, vpool, head_dim: int, v_head_dim: int, page_size: int, scale: float,
+                                     softcap: float = 0.0) -> bool:
+    """Whether ``attention_tcgen05_exact`` takes these operands: bfloat16, one head size of 64 or 128 for keys and values,
+    pages of 8 to 64 keys, rows and pools that start on 16 bytes, a positive scale, a cap of at most 60."""
+    if not (q.dtype is torch.bfloat16 and out.dtype is torch.bfloat16 and kpool.dtype is torch.bfloat16
+            and head_dim == v_head_dim and head_dim in MMA_HEAD_DIMS and scale > 0 and kpool.dim() == 4 == vpool.dim()
+            and kpool.is_contiguous() and vpool.is_contiguous() and kpool.shape == vpool.shape
+            and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
+            and all(t.data_ptr() % 16 == 0 for t in (q, out, kpool, vpool))):
+        return False
+    lib = attention_tcgen05_exact_library()
+    return bool(lib.ie_attention_tcgen05_supports(head_dim, page_size, 0)) and softcap <= lib.ie_attention_tcgen05_max_cap()
+
+
+def attention_tcgen05_exact_error() -> int:
+    """Reads and clears the error word that a timed-out wait of the kernel leaves (0: none)."""
+    return int(attention_tcgen05_exact_library().ie_attention_tcgen05_error())
+
+
+def attention_tcgen05_exact(q, out, kpool, vpool, block_table, q_start, ctx_before, work_req, work_pair0, n_work, n_heads,
+                            n_kv_heads, head_dim, page_size, scale, softcap: float = 0.0, sink: torch.Tensor | None = None,
+                            gate: torch.Tensor | None = None) -> None:
+    """``attention_tcgen05`` with weights in 32 bits (two bfloat16 terms each, both through the tensor cores) and
+    ``attention_general``'s options ``softcap``, ``sink`` and ``gate``; no window."""
+    assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.dtype == torch.int32 and block_table.stride(1) == 1
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (q.shape[0], n_heads))
+    assert sink is None or (sink.dtype is torch.float32 and sink.is_contiguous() and sink.shape == (n_heads,))
+    _check(attention_tcgen05_exact_library().ie_attention_tcgen05_exact(
+        _ptr(q), _ptr(out), _ptr(kpool), _ptr(vpool), _ptr(block_table), _ptr(q_start), _ptr(ctx_before), _ptr(work_req),
+        _ptr(work_pair0), q.stride(0), out.stride(0), block_table.stride(0), n_work, n_heads, n_kv_heads, head_dim,
+        page_size, kpool.shape[0], float(scale), float(softcap), _ptr(sink), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, _stream()),
+        f"attention_tcgen05_exact(head_dim={head_dim}, heads={n_heads}/{n_kv_heads})")
+
+
 def attention_tcgen05_supports(head_dim: int, page_size: int, window) -> bool:
     return bool(attention_tcgen05_library().ie_attention_tcgen05_supports(head_dim, page_size, int(window or 0)))
 

@@ -31,6 +31,7 @@ from .registry import build_position, position_class, register_mixer
 SMALL_REQUEST_TOKENS = 4      # requests that bring at most this many tokens get the split-key rows kernel
 
 
+TCGEN05_MIN_ROWS = 128        # fewer (token, head-in-group) rows than this in every request: smaller tiles waste less
 WIDE_SMALL_MIN_GROUP = 4      # query heads a key head from which decode tokens take the tensor-core kernel too
 
 
@@ -42,8 +43,8 @@ def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: i
     Requests of at most ``SMALL_REQUEST_TOKENS`` tokens (decode tokens): a block per (token, head) whose warps split the
     keys, or, in bfloat16 storage with head sizes that are multiples of 16 and several query heads a key head, the
     tensor-core kernel with the keys split over blocks (every key row is then loaded once for all those heads).  The
-    others (prompt portions), through a work list: the tensor-core kernel under the same conditions, else the float32
-    tile kernel.  ``window``: a query sees itself and the window - 1 keys before it.  ``sink`` (float32 [n_heads]): a
+    others (prompt portions), through a work list: the tcgen05 kernel where it takes the shape (one head size of 64 or 128,
+    every earlier key visible), the tensor-core kernel under the conditions above, else the float32 tile kernel.  ``window``: a query sees itself and the window - 1 keys before it.  ``sink`` (float32 [n_heads]): a
     term exp(sink_h) without key or value in the denominator of head h.  ``softcap`` > 0: scores pass softcap *
     tanh(s / softcap).  ``gate`` ([tokens, n_heads]): head h's output times sigmoid(gate_h)."""
     group = n_heads // n_kv_heads
@@ -76,6 +77,15 @@ def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: i
                                    max_rows, n_heads, n_kv_heads, head_dim, ctx.page_size, window, scale, **extra)
         if n_small == ctx.n_requests:
             return
+    if (ctx.max_q_len * group >= TCGEN05_MIN_ROWS and not window and not chunk and v_row is None
+            and n_v_heads in (None, n_kv_heads)
+            and kernels.attention_tcgen05_exact_supports(q, out, kpool, vpool, head_dim, v_head_dim, ctx.page_size, scale, softcap)):
+        # prompt portions on the tcgen05 tensor cores, with float32 scores and the weights in two bfloat16 terms
+        work_req, work_pair0, n_work = ctx.attention_work(group, kernels.ATTENTION_TCGEN05_ROWS, max_rows if n_small else 0)
+        kernels.attention_tcgen05_exact(q, out, kpool, vpool, kvctx.block_table, ctx.q_start, ctx.ctx_before, work_req,
+                                        work_pair0, n_work, n_heads, n_kv_heads, head_dim, ctx.page_size, scale, softcap,
+                                        sink, gate)
+        return
     if wide:
         # prompt portions in bfloat16 storage: tensor cores, with float32 scores and the weights in two bfloat16 terms
         work_req, work_pair0, n_work = ctx.attention_work(group, kernels.ATTENTION_WIDE_ROWS, max_rows if n_small else 0)

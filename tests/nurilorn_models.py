@@ -71,13 +71,20 @@ NUR_W = _model(300, 128, 1e-5, 4, 3.0, 0.6, 0.3, [
     _att(2, 2, 64, 16, 0.15, 4, _moe(8, 3, 4, 2, 64, 1.1), (10000.0, 64), None, 15.0, True),
     _att(4, 1, 16, 32, 0.3, 2, _moe(8, 4, 2, 2, 32, 0.9), (10000.0, 8), None, None, True),
 ])
+# heads of 64, which the tcgen05 attention takes for portions of enough rows: three query heads a key head under a cap; no
+# cap, a head a key head; a cap beyond what its fixed reference allows, which sends the layer to the other kernels
+NUR_T = _model(200, 144, 1e-5, 2, 2.0, 0.7, 0.5, [
+    _att(3, 1, 64, 64, 0.13, 3, _dense(80, 1.4), (5000.0, 32), (4.0, 64.0, 16.0, 1.0), 25.0, True),
+    _att(2, 1, 64, 64, 0.2, 4, None, (5000.0, 20), None, None, True),
+    _att(1, 1, 64, 64, 0.2, 4, _moe(4, 2, 2, 1, 48, 1.0), None, None, 90.0, True),
+])
 # one mechanism each
 NUR_ATT = _model(120, 48, 1e-5, 2, 2.0, 0.8, 1.0, [_att(6, 3, 12, 8, 0.4, 4, None, (100.0, 8), None, 5.0)])
 NUR_MIX = _model(120, 48, 1e-5, 1, 2.0, 1.0, 1.0, [_att(3, 3, 8, 16, 0.4, 0, None, None, None, None, True) for _ in range(3)])
 NUR_MOE = _model(120, 48, 1e-6, 1, 2.0, 1.0, 1.0, [_att(1, 1, 16, 16, 0.3, 0, _moe(12, 4, 4, 2, 28, 1.0))])
 NUR_DENSE = _model(120, 48, 1e-6, 6, 2.0, 0.5, 2.0, [_att(2, 2, 8, 8, 0.3, 2, _dense(40, 0.5), (100.0, 4))])
 
-MODELS = {"nur_a": NUR_A, "nur_b": NUR_B, "nur_c": NUR_C, "nur_w": NUR_W, "nur_att": NUR_ATT, "nur_mix": NUR_MIX,
+MODELS = {"nur_a": NUR_A, "nur_b": NUR_B, "nur_c": NUR_C, "nur_w": NUR_W, "nur_t": NUR_T, "nur_att": NUR_ATT, "nur_mix": NUR_MIX,
           "nur_moe": NUR_MOE, "nur_dense": NUR_DENSE}
 SEEDS = {name: 81 + i for i, name in enumerate(MODELS)}
 

@@ -312,15 +312,18 @@ def test_experts_with_clamped_branches(dtype, d, ff, experts, top, limit):
     assert limits > 100
 
 
-@pytest.mark.parametrize("kernel", ["rows", "general", "wide", "wide_small"])
-@pytest.mark.parametrize("n_heads, n_k, hd, hdv, cap", [(8, 2, 16, 32, 7.0), (3, 3, 32, 16, 30.0), (4, 1, 48, 48, None), (6, 3, 64, 64, 2.5)])
+@pytest.mark.parametrize("kernel, n_heads, n_k, hd, hdv, cap", [
+    (kernel, *shape) for kernel in ("rows", "general", "wide", "wide_small")
+    for shape in ((8, 2, 16, 32, 7.0), (3, 3, 32, 16, 30.0), (4, 1, 48, 48, None), (6, 3, 64, 64, 2.5))] + [
+    ("tcgen05", *shape) for shape in ((6, 3, 64, 64, 2.5), (8, 2, 64, 64, 30.0), (5, 5, 64, 64, None), (4, 1, 128, 128, 7.0),
+                                      (3, 3, 128, 128, None))])
 def test_a_far_key_stands_out_under_capped_scores(kernel, n_heads, n_k, hd, hdv, cap):
     """One key far back dominates every score it meets (its scores reach the cap); the denominator also holds the term of
     a score of 0, which is most of it for queries whose keys all score far below; every head passes its gate.  Unseen
     pages are poisoned.  float32 kernels in both storage types."""
-    for dt in ([torch.bfloat16] if kernel.startswith("wide") else [torch.float32, torch.bfloat16]):
+    for dt in ([torch.bfloat16] if kernel.startswith(("wide", "tc")) else [torch.float32, torch.bfloat16]):
         g = torch.Generator().manual_seed(13)
-        ps, T, scale, hot = 8, 330, 0.5, 37
+        ps, T, scale, hot = 8, 331, 0.5, 37
         group = n_heads // n_k
         kk = torch.randn(T, n_k, hd, generator=g) * 0.3
         q = torch.randn(T, n_heads, hd, generator=g) * 0.3
@@ -339,7 +342,6 @@ def test_a_far_key_stands_out_under_capped_scores(kernel, n_heads, n_k, hd, hdv,
         perm = torch.randperm(n_pages + 3, generator=g)[:n_pages]
         kpool = torch.full((n_pages + 3, n_k, ps, hd), float("nan"), dtype=dt)
         vpool = torch.full((n_pages + 3, n_k, ps, hdv), float("nan"), dtype=dt)
-        kpool[perm], vpool[perm] = 0, 0
         for t in range(T):
             kpool[perm[t // ps], :, t % ps] = kk[t]
             vpool[perm[t // ps], :, t % ps] = v[t]
@@ -370,11 +372,19 @@ def test_a_far_key_stands_out_under_capped_scores(kernel, n_heads, n_k, hd, hdv,
                     k().attention_wide_small(*args, n_splits, split_keys, scratch, **extra)
                     assert close(out.reshape(R, n_heads, hdv), want[qpos], "bfloat16", rel=2e-2), (splits, n_splits)
         else:
-            rows = k().ATTENTION_WIDE_ROWS if wide else 32
+            rows = {"wide": k().ATTENTION_WIDE_ROWS, "general": 32, "tcgen05": k().ATTENTION_TCGEN05_ROWS}[kernel]
             work = [(0, p0) for p0 in range(0, len(qpos) * group, rows)]
             fn = k().attention_wide if wide else k().attention_general
-            fn(qrows, out, kp, vp, table[None].to(DEV), dev_i32([0, len(qpos)]), dev_i32([30]), dev_i32([x[0] for x in work]),
-               dev_i32([x[1] for x in work]), len(work), n_heads, n_k, hd, ps, None, scale, **extra)
+            if kernel == "tcgen05":
+                assert k().attention_tcgen05_exact_supports(qrows, out, kp, vp, hd, hdv, ps, scale, cap or 0.0)
+                extra.pop("v_head_dim")
+                k().attention_tcgen05_exact(qrows, out, kp, vp, table[None].to(DEV), dev_i32([0, len(qpos)]), dev_i32([30]),
+                                            dev_i32([x[0] for x in work]), dev_i32([x[1] for x in work]), len(work), n_heads, n_k,
+                                            hd, ps, scale, **extra)
+                assert k().attention_tcgen05_exact_error() == 0
+            else:
+                fn(qrows, out, kp, vp, table[None].to(DEV), dev_i32([0, len(qpos)]), dev_i32([30]), dev_i32([x[0] for x in work]),
+                   dev_i32([x[1] for x in work]), len(work), n_heads, n_k, hd, ps, None, scale, **extra)
         got = out.double().cpu().reshape(len(qpos), n_heads, hdv)
         name = "float32" if dt is torch.float32 else "bfloat16"
         for i, p in enumerate(qpos):
@@ -384,32 +394,45 @@ def test_a_far_key_stands_out_under_capped_scores(kernel, n_heads, n_k, hd, hdv,
         assert float(w[:, low].sum(-1).max()) < (0.97 if cap == 2.5 else 0.5)
 
 
-def test_scores_up_to_the_cap_keep_float32_digits():
-    """The tensor-core kernel's form of the hyperbolic tangent against the exact one: two keys, values 0 and 1, so that
-    the output is the logistic of a score (plus the constant), over scores from tiny to far past the cap."""
-    hd = 16
-    for cap in (0.5, 30.0, 400.0):
-        T = 64
+@pytest.mark.parametrize("kernel, hd", [("wide", 16), ("tcgen05", 64), ("tcgen05", 128), ("general", 16)])
+def test_scores_up_to_the_cap_keep_float32_digits(kernel, hd):
+    """The kernels' forms of the hyperbolic tangent against the exact one: n equal keys and values of 1, so that the
+    output is the logistic of a score (plus ln n), over scores from tiny to far past the cap."""
+    for cap in (0.5, 30.0, 60.0, 400.0):
+        T, ps = 160, 16
         x = torch.linspace(-4, 4, T) * cap                       # the uncapped scores
+        x[:64] = torch.linspace(-0.45, 0.45, 64) * cap           # a tile of queries far below the cap
         x[T // 2] = 1e-3 * cap
         q = torch.zeros(T, 1, hd)
         q[:, 0, 0] = x
         q = q.to(torch.bfloat16)
         kk = torch.zeros(T, 1, hd, dtype=torch.bfloat16)
         kk[:, 0, 0] = 1.0
+        pool = lambda t: t.reshape(T // ps, 1, ps, hd).to(DEV)
         v = torch.ones(T, 1, hd, dtype=torch.bfloat16)
         out = torch.empty(T, hd, dtype=torch.bfloat16, device=DEV)
-        k().attention_wide(q.reshape(T, hd).to(DEV), out, kk.reshape(4, 1, 16, hd).to(DEV), v.reshape(4, 1, 16, hd).to(DEV), dev_i32([[0, 1, 2, 3]]),
-                           dev_i32([0, T]), dev_i32([0]), dev_i32([0]), dev_i32([0]), 1, 1, 1, hd, 16, None, 1.0,
-                           sink=torch.zeros(1, device=DEV), softcap=cap)
+        rows = {"wide": k().ATTENTION_WIDE_ROWS, "general": 32, "tcgen05": k().ATTENTION_TCGEN05_ROWS}[kernel]
+        work = list(range(0, T, rows))
+        args = (q.reshape(T, hd).to(DEV), out, pool(kk), pool(v), dev_i32([list(range(T // ps))]), dev_i32([0, T]), dev_i32([0]),
+                dev_i32([0] * len(work)), dev_i32(work), len(work), 1, 1, hd, ps)
+        sink = torch.zeros(1, device=DEV)
+        if kernel == "tcgen05":
+            if cap > 60:
+                assert not k().attention_tcgen05_exact_supports(args[0], out, args[2], args[3], hd, hd, ps, 1.0, cap)
+                with pytest.raises(k().KernelError):
+                    k().attention_tcgen05_exact(*args, 1.0, softcap=cap, sink=sink)
+                continue
+            k().attention_tcgen05_exact(*args, 1.0, softcap=cap, sink=sink)
+            assert k().attention_tcgen05_exact_error() == 0
+        else:
+            (k().attention_wide if kernel == "wide" else k().attention_general)(*args, None, 1.0, softcap=cap, sink=sink)
         s = cap * torch.tanh(q[:, 0, 0].double() / cap)
-        n = torch.arange(1, T + 1, dtype=F)
-        want = torch.sigmoid(s + torch.log(n))                   # n equal scores s beside a score of 0
-        assert torch.allclose(out[:, 0].double().cpu(), want, rtol=5e-3, atol=1e-30), cap
+        want = torch.sigmoid(s + torch.log(torch.arange(1, T + 1, dtype=F)))      # n equal scores s beside a score of 0
+        assert torch.allclose(out[:, 0].double().cpu(), want, rtol=5e-3, atol=1e-30), (kernel, cap)
 
 
 # =============================================================== whole models
-LENGTH = {"nur_a": 97, "nur_b": 70, "nur_c": 131, "nur_w": 190, "nur_att": 75, "nur_mix": 50, "nur_moe": 41, "nur_dense": 60}
+LENGTH = {"nur_a": 97, "nur_b": 70, "nur_c": 131, "nur_w": 190, "nur_t": 280, "nur_att": 75, "nur_mix": 50, "nur_moe": 41, "nur_dense": 60}
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -452,7 +475,7 @@ def test_stream_after_every_layer(tmp_path, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["nur_a", "nur_b", "nur_c", "nur_w"])
+@pytest.mark.parametrize("name", ["nur_a", "nur_b", "nur_c", "nur_w", "nur_t"])
 def test_unequal_requests_in_one_batch_with_pages_and_slots_used_again(tmp_path, name, dtype):
     """Seven requests, at most three live, portions of some beside decoded tokens of others, some left out of a step;
     the pool holds exactly what the fullest moment needs and free pages are filled with NaN."""
@@ -573,7 +596,7 @@ def test_filters_across_the_edges_of_portions_and_pages(tmp_path, dtype, taps):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["nur_att", "nur_w"])
+@pytest.mark.parametrize("name", ["nur_att", "nur_w", "nur_t"])
 def test_a_far_key_is_found(tmp_path, name, dtype):
     """The attention is made sharp; the test first shows that swapping one token 250 and more positions back moves the
     last positions' plain logits, then the engine must agree with the plain model there, in a prompt and decoded (the
@@ -581,7 +604,7 @@ def test_a_far_key_is_found(tmp_path, name, dtype):
     config = copy.deepcopy(MODELS[name])
     for L in config["layers"]:
         L["mixer"]["scale"] *= 2.0
-    folder = make_nurilorn_dir(tmp_path, name, config=config, fix=routers_for(dtype))
+    folder = make_nurilorn_dir(tmp_path, name, config=config, fix=routers_for(dtype) if name != "nur_att" else None)      # it has no router
     cfg, w = plain_inputs(folder)
     toks = steady_tokens(cfg, w, 300, 12)
     ref = reference(w, cfg, toks, dtype)
