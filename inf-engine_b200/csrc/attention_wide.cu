@@ -153,6 +153,33 @@ __device__ __forceinline__ float wide_inv(float l, float m, const float* sink, i
   return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(z * (2.f * LOG2E))));
 }
 
+// raw dot products of a warp's tile to scores in the exponent's base-2 units
+template <int N>
+__device__ __forceinline__ void to_log2_scores(float (&s)[N][4], const WideParams& p) {
+#if IE_AW_CAP
+  float big = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+    big = fmaxf(big, fmaxf(fmaxf(fabsf(s[i][0]), fabsf(s[i][1])), fmaxf(fabsf(s[i][2]), fabsf(s[i][3]))));
+  if (__all_sync(0xffffffffu, big * fabsf(p.cap_in) <= TANH_SMALL)) {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[i][e] = capped_log2(s[i][e], p, true);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[i][e] = capped_log2(s[i][e], p, false);
+  }
+#else
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[i][e] *= p.scale_log2;
+#endif
+}
+
 __device__ __forceinline__ float wide_gate(const WideParams& p, int token, int head) {
   if (p.gate == nullptr) return 1.f;
   return 1.f / (1.f + expf(-to_f32(p.gate[(size_t)token * p.gate_stride + head])));
@@ -263,30 +290,9 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
       }
     }
 
-    // mask, scale, running maximum (exponent units: scale * log2 e is in the multiplier)
+    // scale (and cap), mask, running maximum
+    to_log2_scores<NT_S>(s, p);
     float mx[2] = {-INFINITY, -INFINITY};
-#if IE_AW_CAP
-    {
-      float big = 0.f;
-#pragma unroll
-      for (int nt = 0; nt < NT_S; ++nt)
-        big = fmaxf(big, fmaxf(fmaxf(fabsf(s[nt][0]), fabsf(s[nt][1])), fmaxf(fabsf(s[nt][2]), fabsf(s[nt][3]))));
-      if (__all_sync(0xffffffffu, big * fabsf(p.cap_in) <= TANH_SMALL)) {
-#pragma unroll
-        for (int nt = 0; nt < NT_S; ++nt)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[nt][e] = capped_log2(s[nt][e], p, true);
-      } else {
-#pragma unroll
-        for (int nt = 0; nt < NT_S; ++nt)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[nt][e] = capped_log2(s[nt][e], p, false);
-      }
-    }
-    constexpr float to_log2 = 1.f;
-#else
-    const float to_log2 = p.scale_log2;
-#endif
 #pragma unroll
     for (int nt = 0; nt < NT_S; ++nt) {
 #pragma unroll
@@ -294,7 +300,7 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
         const int h = e >> 1;
         const int kp = kt + nt * 8 + 2 * t4 + (e & 1);
         const bool vis = kp >= lo[h] && kp <= limit[h];
-        const float v = vis ? s[nt][e] * to_log2 : -INFINITY;
+        const float v = vis ? s[nt][e] : -INFINITY;
         s[nt][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -381,6 +387,250 @@ __global__ void __launch_bounds__(THREADS) attention_wide_kernel(WideParams p) {
 #pragma unroll
     for (int i = 0; i < NT_O; ++i)
       *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
+  }
+}
+
+// ------------------------------------------------------------------ a few rows a request (decode tokens)
+// The kernel above gives a tile's rows to its warps, sixteen each; a request whose (token, head-in-group) pairs fit
+// sixteen rows would leave three of four warps idle.  Here the four warps share the rows and split the KEYS: warp w takes
+// the groups of sixteen keys w, w + 4, w + 8, ... of the block's range through a ring of its own in shared memory (no
+// barrier of the block until the end), and the four results are merged in warp order.  Same arithmetic, same options, same
+// partial results for the merge kernel when the keys are split over blocks as well.
+constexpr int RW = THREADS / 32;                      // warps
+constexpr int RK = 16;                                // keys of a group
+constexpr int RSTAGES = (DK + DV <= 256) ? 3 : 2;     // groups on their way a warp
+
+// where the group's keys lie: lane k (and k + 16) of the warp holds key k0 + k's page (-1: read as zeros) and its place there
+__device__ __forceinline__ int2 group_places(const WideParams& p, int k0, int key_end, const int* table, int lane) {
+  const int kp = k0 + (lane & (RK - 1));
+  int2 at = make_int2(-1, 0);
+  if (kp < key_end) {
+    const int logical = kp / p.page_size;
+    at.x = IE_PAGE(table[logical]);
+    at.y = kp - logical * p.page_size;
+  }
+  return at;
+}
+
+__device__ __forceinline__ void load_group(const WideParams& p, bf16* Kg, bf16* Vg, int2 at, int c, int cv, int lane) {
+#pragma unroll
+  for (int i = 0; i < RK * KC / 32; ++i) {
+    const int idx = i * 32 + lane, kk = idx / KC, ch = idx - kk * KC;
+    const int page = __shfl_sync(0xffffffffu, at.x, kk), off = __shfl_sync(0xffffffffu, at.y, kk);
+    bf16* dst = Kg + kk * LDK + ch * 8;
+    if (page >= 0) cp16(dst, p.kpool + (((size_t)page * p.n_kv_heads + c) * p.page_size + off) * DK + ch * 8);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+  }
+  if (p.alias) return;
+#pragma unroll
+  for (int i = 0; i < RK * VC / 32; ++i) {
+    const int idx = i * 32 + lane, kk = idx / VC, ch = idx - kk * VC;
+    const int page = __shfl_sync(0xffffffffu, at.x, kk), off = __shfl_sync(0xffffffffu, at.y, kk);
+    bf16* dst = Vg + kk * LDV + ch * 8;
+    if (page >= 0) cp16(dst, p.vpool + (((size_t)page * p.n_v_heads + cv) * p.page_size + off) * p.v_row + ch * 8);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+  }
+}
+
+__global__ void __launch_bounds__(THREADS) attention_wide_rows_kernel(WideParams p) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  pdl_trigger();
+  pdl_wait();
+  const int ring_group = RK * (LDK + (p.alias ? 0 : LDV));
+  bf16* Qs = reinterpret_cast<bf16*>(smem_raw);       // [16][LDK]
+  bf16* rings = Qs + 16 * LDK;                        // [RW][RSTAGES][RK][LDK] then [RK][LDV]
+  float* merged = reinterpret_cast<float*>(rings);    // afterwards: [RW][16][DV], the rings being used up
+  __shared__ float s_m[RW][16], s_l[RW][16];
+
+  const int r_id = blockIdx.x, c = blockIdx.y;
+  const int group = p.n_heads / p.n_kv_heads;
+  const int cv = c / (p.n_kv_heads / p.n_v_heads);
+  const int q0 = p.q_start[r_id];
+  const int n_pairs = (p.q_start[r_id + 1] - q0) * group;
+  if (n_pairs > p.max_rows || n_pairs <= 0) return;
+  const int ctx = p.ctx_before[r_id];
+  const int* table = p.block_table + (size_t)r_id * p.table_stride;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+
+  int limit[2], lo[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int pr = g + 8 * h;
+    limit[h] = -1;
+    lo[h] = 0;
+    if (pr < n_pairs) {
+      limit[h] = ctx + pr / group;
+      int first = p.window > 0 ? max(0, limit[h] - p.window + 1) : 0;
+      if (p.chunk > 0) first = max(first, (limit[h] / p.chunk) * p.chunk);
+      lo[h] = first;
+    }
+  }
+  const int key_end = ctx + (n_pairs - 1) / group + 1;
+  int key_begin = 0;
+  if (p.window > 0) key_begin = max(0, ctx - p.window + 1);
+  if (p.chunk > 0) key_begin = max(key_begin, (ctx / p.chunk) * p.chunk);
+  key_begin = (key_begin / BN) * BN;
+  int k_lo = key_begin, k_hi = key_end;
+  if (p.n_splits > 1) {
+    k_lo = key_begin + (int)blockIdx.z * p.split_keys;
+    k_hi = min(key_end, k_lo + p.split_keys);
+  }
+
+  bf16* ring = rings + (size_t)warp * RSTAGES * ring_group;
+  const int n_groups = k_lo < k_hi ? (k_hi - k_lo + RK - 1) / RK : 0;
+  const int mine = n_groups > warp ? (n_groups - warp + RW - 1) / RW : 0;
+  auto key_of = [&](int i) { return k_lo + (warp + i * RW) * RK; };
+  int2 at[RSTAGES];                                     // page lookups run ahead of the copies that need them
+#pragma unroll
+  for (int i = 0; i < RSTAGES; ++i) at[i] = group_places(p, key_of(i), k_hi, table, lane);
+#pragma unroll
+  for (int i = 0; i < RSTAGES - 1; ++i) {
+    if (i < mine) load_group(p, ring + i * ring_group, ring + i * ring_group + RK * LDK, at[i], c, cv, lane);
+    cp_commit();
+  }
+  int2 next_at = at[RSTAGES - 1];
+  // the rows' queries
+  for (int idx = tid; idx < 16 * KC; idx += THREADS) {
+    const int r = idx / KC, ch = idx - r * KC;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (r < n_pairs) {
+      const int t = r / group, j = r - t * group;
+      v = *reinterpret_cast<const uint4*>(p.q + (size_t)(q0 + t) * p.q_stride + (size_t)(c * group + j) * DK + ch * 8);
+    }
+    *reinterpret_cast<uint4*>(Qs + r * LDK + ch * 8) = v;
+  }
+  __syncthreads();
+
+  float o[NT_O][4];
+#pragma unroll
+  for (int i = 0; i < NT_O; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  const int ldv = p.alias ? LDK : LDV;
+  for (int i = 0; i < mine; ++i) {
+    {
+      const int nx = i + RSTAGES - 1;
+      bf16* dst = ring + (nx % RSTAGES) * ring_group;
+      if (nx < mine) load_group(p, dst, dst + RK * LDK, next_at, c, cv, lane);
+      cp_commit();
+      next_at = group_places(p, key_of(nx + 1), k_hi, table, lane);
+      cp_wait<RSTAGES - 1>();
+    }
+    __syncwarp();
+    const bf16* Kt = ring + (i % RSTAGES) * ring_group;
+    const bf16* Vt = p.alias ? Kt : Kt + RK * LDK;
+    const int kt = key_of(i);
+    float s[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < KSTEPS; ++ks) {
+      unsigned a[4], b[4];
+      ldsm4(a, Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * LDK + ks * 16 + (lane >> 4) * 8);
+      ldsm4(b, Kt + ((lane & 7) + (lane >> 4) * 8) * LDK + ks * 16 + ((lane >> 3) & 1) * 8);
+      mma16816(s[0], a, b[0], b[1]);
+      mma16816(s[1], a, b[2], b[3]);
+    }
+    to_log2_scores<2>(s, p);
+    float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int h = e >> 1;
+        const int kp = kt + n * 8 + 2 * t4 + (e & 1);
+        const float v = (kp >= lo[h] && kp <= limit[h] && kp < k_hi) ? s[n][e] : -INFINITY;
+        s[n][e] = v;
+        mx[h] = fmaxf(mx[h], v);
+      }
+    }
+    float alpha[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+      mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+      const float m_new = fmaxf(m_run[h], mx[h]);
+      alpha[h] = m_new == -INFINITY ? 1.f : exp2f(m_run[h] - m_new);
+      m_run[h] = m_new;
+      l_run[h] *= alpha[h];
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int h = e >> 1;
+        const float pv = m_run[h] == -INFINITY ? 0.f : exp2f(s[n][e] - m_run[h]);
+        s[n][e] = pv;
+        l_run[h] += pv;
+      }
+    }
+#pragma unroll
+    for (int d = 0; d < NT_O; ++d) {
+      o[d][0] *= alpha[0]; o[d][1] *= alpha[0];
+      o[d][2] *= alpha[1]; o[d][3] *= alpha[1];
+    }
+    unsigned ah[4], al[4];
+    split2(s[0][0], s[0][1], ah[0], al[0]);
+    split2(s[0][2], s[0][3], ah[1], al[1]);
+    split2(s[1][0], s[1][1], ah[2], al[2]);
+    split2(s[1][2], s[1][3], ah[3], al[3]);
+#pragma unroll
+    for (int dp = 0; dp < NT_O / 2; ++dp) {
+      unsigned b[4];
+      ldsm4_t(b, Vt + ((lane & 7) + ((lane >> 3) & 1) * 8) * ldv + dp * 16 + (lane >> 4) * 8);
+      mma16816(o[2 * dp], ah, b[0], b[1]);
+      mma16816(o[2 * dp], al, b[0], b[1]);
+      mma16816(o[2 * dp + 1], ah, b[2], b[3]);
+      mma16816(o[2 * dp + 1], al, b[2], b[3]);
+    }
+    __syncwarp();                                      // the group is used up before the load after next overwrites it
+  }
+  cp_wait<0>();
+  __syncthreads();                                     // the rings become the place where the warps' results meet
+
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    float l = l_run[h];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    const int r = g + 8 * h;
+    if (t4 == 0) {
+      s_m[warp][r] = m_run[h];
+      s_l[warp][r] = l;
+    }
+    float* dst = merged + ((size_t)warp * 16 + r) * DV + 2 * t4;
+#pragma unroll
+    for (int i = 0; i < NT_O; ++i) *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
+  }
+  __syncthreads();
+  const int rows = min(16, n_pairs);
+  for (int idx = tid; idx < rows * (DV / 2); idx += THREADS) {
+    const int r = idx / (DV / 2), d = (idx - r * (DV / 2)) * 2;
+    float m = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < RW; ++w) m = fmaxf(m, s_m[w][r]);
+    float l = 0.f;
+    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < RW; ++w) {
+      const float f = s_m[w][r] == -INFINITY ? 0.f : exp2f(s_m[w][r] - m);
+      const float2 v = *reinterpret_cast<const float2*>(merged + ((size_t)w * 16 + r) * DV + d);
+      l = fmaf(s_l[w][r], f, l);
+      acc.x = fmaf(v.x, f, acc.x);
+      acc.y = fmaf(v.y, f, acc.y);
+    }
+    if (p.n_splits > 1) {
+      const size_t row = (((size_t)blockIdx.x * p.n_kv_heads + c) * p.n_splits + blockIdx.z) * BM + r;
+      if (d == 0) {
+        p.part_ml[row * 2] = m;
+        p.part_ml[row * 2 + 1] = l;
+      }
+      *reinterpret_cast<float2*>(p.part_o + row * DV + d) = acc;
+    } else {
+      const int t = r / group, j = r - t * group;
+      const float inv = wide_inv(l, m, p.sink, c * group + j) * wide_gate(p, q0 + t, c * group + j);
+      *reinterpret_cast<__nv_bfloat162*>(p.out + (size_t)(q0 + t) * p.out_stride + (size_t)(c * group + j) * DV + d) =
+          __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
+    }
   }
 }
 
@@ -528,11 +778,17 @@ extern "C" int ie_attention_wide_small(const void* q, void* out, const void* kpo
   const size_t n_parts = (size_t)n_requests * p.tiles * n_kv_heads * n_splits;
   p.part_o = scratch;
   p.part_ml = scratch != nullptr ? scratch + n_parts * BM * DV : nullptr;
-  const size_t smem = wide_smem(p);
-  cudaError_t e = cudaFuncSetAttribute(attention_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const bool few = max_rows <= 16;                     // the warps of a block share the rows and split the keys
+  size_t smem = wide_smem(p);
+  if (few) {
+    const size_t ring = sizeof(bf16) * RW * RSTAGES * RK * (size_t)(LDK + (p.alias ? 0 : LDV)), merged = sizeof(float) * RW * 16 * DV;
+    smem = sizeof(bf16) * 16 * LDK + (ring > merged ? ring : merged);
+  }
+  auto kernel = few ? attention_wide_rows_kernel : attention_wide_kernel;
+  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const dim3 grid(n_requests * p.tiles, n_kv_heads, n_splits);
-  int st = launch_k(attention_wide_kernel, grid, THREADS, smem, stream, p);
+  int st = launch_k(kernel, grid, THREADS, smem, stream, p);
   if (st != IE_OK || n_splits == 1) return st;
   return launch_k(attention_wide_merge_kernel, dim3(grid.x, grid.y, BM / MERGE_ROWS), THREADS, 0, stream, p);
 }

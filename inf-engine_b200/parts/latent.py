@@ -32,7 +32,6 @@ SMALL_REQUEST_TOKENS = 4      # requests that bring at most this many tokens get
 
 
 TCGEN05_MIN_ROWS = 128        # fewer (token, head-in-group) rows than this in every request: smaller tiles waste less
-WIDE_SMALL_MIN_GROUP = 4      # query heads a key head from which decode tokens take the tensor-core kernel too
 
 
 def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int,
@@ -41,24 +40,25 @@ def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: i
                    gate: torch.Tensor | None = None) -> None:
     """Causal attention of the step's queries over the paged keys with float32 scores, maxima, weights and sums.
     Requests of at most ``SMALL_REQUEST_TOKENS`` tokens (decode tokens): a block per (token, head) whose warps split the
-    keys, or, in bfloat16 storage with head sizes that are multiples of 16 and several query heads a key head, the
-    tensor-core kernel with the keys split over blocks (every key row is then loaded once for all those heads).  The
+    keys, or, in bfloat16 storage with head sizes that are multiples of 16, the tensor-core kernel with the keys split
+    over warps and blocks (every key row is then loaded once for all query heads of its key head).  The
     others (prompt portions), through a work list: the tcgen05 kernel where it takes the shape (one head size of 64 or 128,
     every earlier key visible), the tensor-core kernel under the conditions above, else the float32 tile kernel.  ``window``: a query sees itself and the window - 1 keys before it.  ``sink`` (float32 [n_heads]): a
     term exp(sink_h) without key or value in the denominator of head h.  ``softcap`` > 0: scores pass softcap *
     tanh(s / softcap).  ``gate`` ([tokens, n_heads]): head h's output times sigmoid(gate_h)."""
     group = n_heads // n_kv_heads
-    max_rows = SMALL_REQUEST_TOKENS * group
     if ctx.max_q_len <= SMALL_REQUEST_TOKENS:
-        n_small = ctx.n_requests
+        n_small, most = ctx.n_requests, ctx.max_q_len
     else:
-        n_small = sum(1 for n in ctx.host["q_lens"] if n <= SMALL_REQUEST_TOKENS)
+        small = [n for n in ctx.host["q_lens"] if n <= SMALL_REQUEST_TOKENS]
+        n_small, most = len(small), max(small, default=0)
+    max_rows = most * group          # what the small requests bring at most; every other request brings more
     extra = dict(v_head_dim=v_head_dim, chunk=chunk or 0, n_v_heads=n_v_heads, v_row=v_row, sink=sink, softcap=softcap,
                  gate=gate)
     wide = (kpool.dtype is torch.bfloat16 and kernels.attention_wide_supports(q, out, head_dim, v_head_dim, v_row)
             and kpool.data_ptr() % 16 == 0 and vpool.data_ptr() % 16 == 0)
     if n_small:
-        if wide and group >= WIDE_SMALL_MIN_GROUP:
+        if wide:
             rows = kernels.ATTENTION_WIDE_ROWS
             # the longest run of keys a small request may see, from the tile boundary below its first key
             keys = min(ctx.keys_cap, chunk + SMALL_REQUEST_TOKENS) if chunk else ctx.keys_cap
