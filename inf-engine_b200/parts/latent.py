@@ -12,10 +12,9 @@ query heads over 2 x kv_heads key heads and kv_heads value heads.  The query row
 (``[kv head, map, head in group]``) so that the query heads of one key head lie side by side, as the attention
 kernels expect; a kernel then forms ``a1 - lambda a2``, norms it, and applies the output gate.
 
-Both keep scores, maxima, weights and sums in float32 whatever the storage type: a block per (token, head) whose
-warps split the keys for requests that bring a few tokens; for prompt portions the tensor-core kernel with float32
-scores (``kernels.attention_wide``: bfloat16 storage, head sizes that are multiples of 16) or else the float32 tile
-kernel on CUDA cores.
+Both keep scores, maxima, weights and sums in float32 whatever the storage type (``attend_float32``): the tensor-core
+kernels with float32 scores for bfloat16 storage and head sizes that they take, split over the keys for requests that
+bring a few tokens; else the float32 kernels on CUDA cores.
 """
 
 from __future__ import annotations
@@ -29,8 +28,6 @@ from .linear import Linear, stack_rows
 from .registry import build_position, position_class, register_mixer
 
 SMALL_REQUEST_TOKENS = 4      # requests that bring at most this many tokens get the split-key rows kernel
-
-
 TCGEN05_MIN_ROWS = 128        # fewer (token, head-in-group) rows than this in every request: smaller tiles waste less
 
 
@@ -43,8 +40,8 @@ def attend_float32(q, out, kpool, vpool, ctx, kvctx, n_heads: int, n_kv_heads: i
     keys, or, in bfloat16 storage with head sizes that are multiples of 16, the tensor-core kernel with the keys split
     over warps and blocks (every key row is then loaded once for all query heads of its key head).  The
     others (prompt portions), through a work list: the tcgen05 kernel where it takes the shape (one head size of 64 or 128,
-    every earlier key visible), the tensor-core kernel under the conditions above, else the float32 tile kernel.  ``window``: a query sees itself and the window - 1 keys before it.  ``sink`` (float32 [n_heads]): a
-    term exp(sink_h) without key or value in the denominator of head h.  ``softcap`` > 0: scores pass softcap *
+    every earlier key visible), the tensor-core kernel under the conditions above, else the float32 tile kernel.
+    ``window``: a query sees itself and the window - 1 keys before it.  ``sink`` (float32 [n_heads]): a term exp(sink_h) without key or value in the denominator of head h.  ``softcap`` > 0: scores pass softcap *
     tanh(s / softcap).  ``gate`` ([tokens, n_heads]): head h's output times sigmoid(gate_h)."""
     group = n_heads // n_kv_heads
     if ctx.max_q_len <= SMALL_REQUEST_TOKENS:
