@@ -4,6 +4,7 @@ from .gavatar import GavatarConfig
 from .kipezen import KipezenConfig
 from .llama import ConfigError, LlamaConfig
 from .nurilorn import NurilornConfig
+from .nurasun import NurasunConfig
 from .registry import (
     ARCHITECTURES,
     Architecture,
@@ -20,6 +21,7 @@ from .spec import (
     ConvAttentionSpec,
     DifferentialAttentionSpec,
     LatentAttentionSpec,
+    MLPSpec,
     MinGRUSpec,
     ReinjectDecoderSpec,
     YarnScaling,
@@ -41,4 +43,5 @@ from .spec import (
     RoutedExpertsSpec,
     ScheduleEntry,
     ShortConvSpec,
+    TiedAttentionSpec,
 )

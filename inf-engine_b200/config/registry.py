@@ -138,3 +138,11 @@ def _nurilorn(d: dict):
 
 
 register_architecture("Nurilorn", _nurilorn)
+
+
+def _nurasun(d: dict):
+    from .nurasun import NurasunConfig
+    return NurasunConfig.from_dict(d)
+
+
+register_architecture("Nurasun", _nurasun)

@@ -30,15 +30,18 @@ class RopeScaling:
 class NormSpec:
     """A normalisation over the last axis."""
 
-    kind: str          # "rmsnorm" | "layernorm" | "grouped_rmsnorm"
+    kind: str          # "rmsnorm" | "layernorm" | "grouped_rmsnorm" | "tanh_norm"
     size: int
     eps: float
     weight: str        # tensor name of the gain
-    bias: str | None = None   # tensor name of the additive term ("layernorm")
+    bias: str | None = None   # tensor name of the additive term ("layernorm", "tanh_norm")
     unit_offset: bool = False  # "rmsnorm": the tensor is stored around zero and the multiplier is 1 + weight
     scalar: bool = False       # "rmsnorm": the tensor is ONE number (shape ()), the multiplier of every coordinate
     groups: int = 1            # "grouped_rmsnorm": the row is split into this many equal parts, each normed by itself
     out_scale: float = 1.0     # "grouped_rmsnorm": a constant multiplier of the normed row
+    # "tanh_norm" (dynamic tanh): tanh(alpha x) * weight + bias, coordinate by coordinate; ``alpha`` names the tensor of
+    # the one number (shape ()); no statistic of the row enters and ``eps`` is not used
+    alpha: str | None = None
 
 
 @dataclass(frozen=True)
@@ -171,6 +174,31 @@ class LatentAttentionSpec(MixerSpec):
     sink: str | None = None        # tensor [n_heads]: exp(sink_h) joins the softmax's denominator of head h: a learned
                                    # logit beside the keys' scores that ``scale`` does not multiply and that weighs nothing
     head_gate: str | None = None   # tensor [n_heads, hidden]: head h's output is multiplied by sigmoid(head_gate x)_h
+    # ``down_proj`` "": the layer compresses nothing itself and reads the vectors that another run's cache holds (the
+    # schedule entry's ``cache_from``), with its own queries, expansions and scale.
+
+
+@dataclass(frozen=True)
+class TiedAttentionSpec(MixerSpec):
+    """Causal grouped-query softmax attention without a value projection: the values are the projected keys (with their
+    bias) before their rotation.
+
+    q, k = q_proj x, k_proj x (+ biases); v = k; then ``position`` ("rotary_partial" or "none") turns the first dimensions
+    of every query and key head.  score = q . k * scale over the earlier keys, of the query's own chunk of ``chunk``
+    positions only when that is given; ordinary softmax; ``o_proj`` on the concatenated heads."""
+
+    hidden: int = 0
+    n_heads: int = 0
+    n_kv_heads: int = 0
+    head_dim: int = 0
+    scale: float = 1.0
+    position: PositionSpec = PositionSpec(kind="none")
+    chunk: int | None = None
+    q_proj: str = ""
+    k_proj: str = ""
+    q_bias: str | None = None
+    k_bias: str | None = None
+    o_proj: str = ""
 
 
 @dataclass(frozen=True)
@@ -441,7 +469,8 @@ class FeedForwardSpec:
 @dataclass(frozen=True)
 class GatedMLPSpec(FeedForwardSpec):
     """``down(act(gate(x)) * (up(x) + up_offset))``.  ``activation`` "silu": g sigmoid(g).  "clamped_swish": with
-    g' = min(g, act_limit) and up clamped to [-act_limit, act_limit], g' sigmoid(act_alpha g')."""
+    g' = min(g, act_limit) and up clamped to [-act_limit, act_limit], g' sigmoid(act_alpha g').  "gelu_tanh": the tanh
+    form of gelu, g / 2 (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3)))."""
 
     hidden: int = 0
     intermediate: int = 0
@@ -450,6 +479,17 @@ class GatedMLPSpec(FeedForwardSpec):
     act_limit: float = 0.0
     up_offset: float = 0.0
     gate_proj: str = ""
+    up_proj: str = ""
+    down_proj: str = ""
+
+
+@dataclass(frozen=True)
+class MLPSpec(FeedForwardSpec):
+    """``down(act(up(x)))``: a feed-forward without a gate.  ``activation`` "relu2": max(z, 0)^2."""
+
+    hidden: int = 0
+    intermediate: int = 0
+    activation: str = "relu2"
     up_proj: str = ""
     down_proj: str = ""
 
@@ -479,7 +519,8 @@ class RoutedExpertsSpec(FeedForwardSpec):
     experts of the ``keep_groups`` best groups can be chosen.  The ``top`` largest choice scores among them are
     taken; their weights are their s divided by the sum of those (+ ``weight_eps``), times ``route_scale``.  The
     output is the weighted sum of the chosen experts' ``down(silu(gate x) * up x)``.  ``shared`` (optional) is a
-    dense expert that every token runs; it is added times sigmoid(shared_gate x), one number a token."""
+    dense expert that every token runs (of any feed-forward kind); it is added times sigmoid(shared_gate x), one number
+    a token, or as it is without a ``shared_gate``."""
 
     hidden: int = 0
     intermediate: int = 0
@@ -492,7 +533,7 @@ class RoutedExpertsSpec(FeedForwardSpec):
     router: str = ""
     correction: str | None = None
     expert_prefix: str = ""        # expert e's tensors are <prefix><e>.gate / .up / .down
-    shared: GatedMLPSpec | None = None
+    shared: FeedForwardSpec | None = None
     shared_gate: str | None = None
     # ``score`` "softmax_top": the logits are router x + ``router_bias`` (float32); the ``top`` largest are chosen (no
     # groups, no correction) and their weights are the softmax over the chosen logits alone, times ``route_scale``.
@@ -500,7 +541,9 @@ class RoutedExpertsSpec(FeedForwardSpec):
     score: str = "sigmoid"
     router_bias: str | None = None
     group_score: str = "top2_sum"  # a group's score: the sum of its two largest choice scores, or "max": the largest
-    # the experts' activation, as ``GatedMLPSpec`` states it
+    # the experts' activation, as ``GatedMLPSpec`` states it; ``gated`` False: experts are ``down(act(up x))`` without a
+    # gate tensor, with an activation of ``MLPSpec``
+    gated: bool = True
     activation: str = "silu"
     act_alpha: float = 1.0
     act_limit: float = 0.0
@@ -535,6 +578,8 @@ class BlockSpec:
     residual_mult: float = 1.0
     mixer_scale: str | None = None
     ff_scale: str | None = None
+    # "parallel": x += residual_mult * (mixer(h) + ff(h)) with h = mixer_norm(x): one norm, whose output both sublayers
+    # read (``ff_norm`` is None)
 
 
 @dataclass(frozen=True)
@@ -566,6 +611,7 @@ class ModelSpec:
     optional_tensors: tuple[str, ...] = field(default_factory=tuple)  # present-but-unused names tolerated
     kind: str = "decoder"                    # which registered top level puts the parts together
     embedding_scale: float = 1.0             # multiplier of the token embedding
+    logit_softcap: float | None = None       # logits <- cap * tanh(logits / cap)
 
 
 @dataclass(frozen=True)

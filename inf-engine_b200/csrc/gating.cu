@@ -4,8 +4,10 @@
 // gated_residual_add:  residual += sigmoid(gate_pre + bias) * y          (residual float32; a gate per coordinate)
 // scale_rows:          x *= scale, and a copy of the result where asked   (a scaled embedding that is used again later)
 // glu_act:             out = act(g) * (u + up_offset) over rows that hold gate and up side by side or alternating:
-//                      kind 0: g * sigmoid(g);  kind 1: g' * sigmoid(alpha g') with g' = min(g, limit) and u clamped to
-//                      [-limit, limit]
+//                      kind 0: g * sigmoid(g);  kind 1: g' * sigmoid(alpha g' + cubic g'^3) with g' = min(g, limit) and u
+//                      clamped to [-limit, limit] (the tanh form of gelu is such a one: 1/2 (1 + tanh z) = sigmoid(2 z))
+// relu2:               out = max(x, 0)^2
+// softcap:             x <- cap * tanh(x / cap), in place
 // mingru_scan:         z = sigmoid(z_pre + z_bias), u = u_pre + u_bias, candidate = u + 1/2 (u >= 0) | sigmoid(u) (u < 0)
 //                      S <- S + z (candidate - S)   [= (1 - z) S + z candidate],  out = S * silu(g_pre)
 //                      per channel, over each request's tokens of the step in order, from the float32 state of the
@@ -104,7 +106,7 @@ extern "C" int ie_scale_rows(float* x, float* keep, float scale, int n_rows, int
 
 template <typename T>
 __global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, int inter, int in_stride, size_t total,
-                               int interleaved, int kind, float alpha, float limit, float up_offset) {
+                               int interleaved, int kind, float alpha, float limit, float up_offset, float cubic) {
   pdl_trigger();
   pdl_wait();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -117,7 +119,7 @@ __global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, in
   if (kind == 1) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
-    a = g * sigmoid_f(alpha * g);
+    a = g * sigmoid_f(g * fmaf(cubic * g, g, alpha));
   } else {
     a = g * sigmoid_f(g);
   }
@@ -126,7 +128,8 @@ __global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, in
 
 // bfloat16, eight outputs a thread (inter and the row stride multiples of 8, rows that start on 16 bytes)
 __global__ void glu_act_bf16_vec_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, int inter, int in_stride,
-                                        size_t total8, int interleaved, int kind, float alpha, float limit, float up_offset) {
+                                        size_t total8, int interleaved, int kind, float alpha, float limit, float up_offset,
+                                        float cubic) {
   pdl_trigger();
   pdl_wait();
   const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -156,7 +159,7 @@ __global__ void glu_act_bf16_vec_kernel(const bf16* __restrict__ in, bf16* __res
     if (kind == 1) {
       gg = fminf(gg, limit);
       uu = fminf(fmaxf(uu, -limit), limit);
-      act = gg * sigmoid_f(alpha * gg);
+      act = gg * sigmoid_f(gg * fmaf(cubic * gg, gg, alpha));
     } else {
       act = gg * sigmoid_f(gg);
     }
@@ -170,23 +173,63 @@ __global__ void glu_act_bf16_vec_kernel(const bf16* __restrict__ in, bf16* __res
 }
 
 extern "C" int ie_glu_act(const void* in, void* out, int n_rows, int inter, int in_stride, int interleaved, int kind,
-                          float alpha, float limit, float up_offset, int act_dtype, cudaStream_t stream) {
+                          float alpha, float limit, float up_offset, float cubic, int act_dtype, cudaStream_t stream) {
   const size_t total = (size_t)n_rows * inter;
   if (total == 0) return IE_OK;
   if (kind < 0 || kind > 1) return IE_BAD_SIZE;
   if (act_dtype == IE_BF16 && inter % 8 == 0 && in_stride % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
     const size_t total8 = total / 8;
     return launch_k(glu_act_bf16_vec_kernel, (unsigned)((total8 + 255) / 256), 256, 0, stream, (const bf16*)in, (bf16*)out,
-                    inter, in_stride, total8, interleaved, kind, alpha, limit, up_offset);
+                    inter, in_stride, total8, interleaved, kind, alpha, limit, up_offset, cubic);
   }
   const unsigned blocks = (unsigned)((total + 255) / 256);
   if (act_dtype == IE_F32)
     return launch_k(glu_act_kernel<float>, blocks, 256, 0, stream, (const float*)in, (float*)out, inter, in_stride, total,
-                    interleaved, kind, alpha, limit, up_offset);
+                    interleaved, kind, alpha, limit, up_offset, cubic);
   if (act_dtype == IE_BF16)
     return launch_k(glu_act_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)in, (bf16*)out, inter, in_stride, total,
-                    interleaved, kind, alpha, limit, up_offset);
+                    interleaved, kind, alpha, limit, up_offset, cubic);
   return IE_BAD_DTYPE;
+}
+
+// ------------------------------------------------------------------ the square of relu, a cap by a hyperbolic tangent
+// out[n, j] = max(in[n, j], 0)^2 over rows with a stride
+template <typename T>
+__global__ void relu2_kernel(const T* __restrict__ in, int in_stride, T* __restrict__ out, int out_stride, int cols,
+                             size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const size_t n = i / cols, j = i - n * cols;
+  const float v = fmaxf(to_f32(in[n * in_stride + j]), 0.f);
+  out[n * out_stride + j] = from_f32<T>(v * v);
+}
+
+extern "C" int ie_relu2(const void* in, int in_stride, void* out, int out_stride, int n_rows, int cols, int act_dtype,
+                        cudaStream_t stream) {
+  const size_t total = (size_t)n_rows * cols;
+  if (total == 0) return IE_OK;
+  const unsigned blocks = (unsigned)((total + 255) / 256);
+  if (act_dtype == IE_F32)
+    return launch_k(relu2_kernel<float>, blocks, 256, 0, stream, (const float*)in, in_stride, (float*)out, out_stride, cols, total);
+  if (act_dtype == IE_BF16)
+    return launch_k(relu2_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)in, in_stride, (bf16*)out, out_stride, cols, total);
+  return IE_BAD_DTYPE;
+}
+
+// x <- cap * tanh(x / cap), float32, in place
+__global__ void softcap_kernel(float* __restrict__ x, float cap, size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < total) x[i] = cap * tanhf(x[i] / cap);
+}
+
+extern "C" int ie_softcap(float* x, float cap, size_t total, cudaStream_t stream) {
+  if (total == 0) return IE_OK;
+  if (!(cap > 0.f)) return IE_BAD_SIZE;
+  return launch_k(softcap_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, x, cap, total);
 }
 
 #define MG_UNROLL 4

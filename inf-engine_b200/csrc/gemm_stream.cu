@@ -12,6 +12,8 @@
 //             RESIDUAL   residual[M,N] += product in float32 (engine/llama_block.py:54,62)
 //             SILU_MUL   weight rows alternate gate_j, up_j; out[M, N/2] =
 //                        silu(gate_j) * up_j in float32 (engine/llama_mlp.py:30-32)
+//             GLU        the same with the activation's constants as parameters
+//             RELU2      out[M, N] = max(product, 0)^2
 //
 // At these sizes the product is bound by reading W once from HBM.  Every lane
 // loads 16 bytes of a weight row straight from global memory into the B
@@ -23,7 +25,7 @@
 namespace {
 
 enum { PRO_PLAIN = 0, PRO_NORM = 1 };
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SILU_MUL = 3 };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SILU_MUL = 3, EPI_RELU2 = 5, EPI_GLU = 6 };
 
 constexpr int GS_WARPS = 8;
 constexpr int GS_THREADS = GS_WARPS * 32;
@@ -37,7 +39,21 @@ struct StreamParams {
   int M, N, K, lda, ldw, ldc;
   int gain_is_f32;
   float eps;
+  float act_alpha, act_limit, act_offset, act_cubic;   // GLU
 };
+
+// the gated activation of the GLU epilogue: g' sigmoid(alpha g' + cubic g'^3) (u' + offset), g' = min(g, limit) and u' = u
+// clamped to [-limit, limit]
+template <typename P>
+__device__ __forceinline__ float stream_glu(const P& p, float g, float u) {
+  g = fminf(g, p.act_limit);
+  u = fminf(fmaxf(u, -p.act_limit), p.act_limit) + p.act_offset;
+  return g / (1.f + expf(-g * fmaf(p.act_cubic * g, g, p.act_alpha))) * u;
+}
+__device__ __forceinline__ float stream_relu2(float v) {
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
 
 // Weights are read once a step and are far larger than L2: "evict first" keeps the stream from pushing out
 // what the step reads again and again (activations, norm gains, the kernels' own code).
@@ -225,7 +241,11 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_stream_kernel(StreamParams p)
       v1 *= inv;
     }
     const bool has1 = n + 1 < p.N;
-    if (EPI == EPI_BF16) {
+    if (EPI == EPI_RELU2) {
+      v0 = stream_relu2(v0);
+      v1 = stream_relu2(v1);
+    }
+    if (EPI == EPI_BF16 || EPI == EPI_RELU2) {
       bf16* c = (bf16*)p.C + (size_t)m * p.ldc + n;
       if (has1 && ((((uintptr_t)c) & 3) == 0)) *reinterpret_cast<uint32_t*>(c) = pack2(v0, v1);
       else { c[0] = __float2bfloat16_rn(v0); if (has1) c[1] = __float2bfloat16_rn(v1); }
@@ -237,6 +257,8 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_stream_kernel(StreamParams p)
       float* c = (float*)p.C + (size_t)m * p.ldc + n;
       c[0] += v0;
       if (has1) c[1] += v1;
+    } else if (EPI == EPI_GLU) {
+      ((bf16*)p.C)[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn(stream_glu(p, v0, v1));
     } else {  // EPI_SILU_MUL: v0 = gate_j, v1 = up_j, j = n / 2
       const float sg = 1.f / (1.f + expf(-v0));
       ((bf16*)p.C)[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn((v0 * sg) * v1);
@@ -273,20 +295,23 @@ int dispatch(const StreamParams& p, int nt, cudaStream_t stream) {
 }  // namespace
 
 // pro: 0 plain bf16 A, 1 float32 residual with fused RMSNorm (gain, eps, optional row_index)
-// epi: 0 bf16 out, 1 float32 out, 2 residual +=, 3 silu(gate)*up over interleaved weight rows
+// epi: 0 bf16 out, 1 float32 out, 2 residual +=, 3 silu(gate)*up over interleaved weight rows, 5 max(., 0)^2 (bf16 out),
+//      6 the gated activation with the constants act_* over interleaved weight rows
 // nt:  8*nt weight rows per block (1, 2 or 4)
 extern "C" int ie_gemm_stream(const void* A, const void* W, void* C, const void* gain, int gain_dtype,
                               const int* row_index, int M, int N, int K, int lda, int ldw, int ldc, float eps,
-                              int pro, int epi, int nt, cudaStream_t stream) {
+                              int pro, int epi, int nt, float act_alpha, float act_limit, float act_offset,
+                              float act_cubic, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return IE_OK;
   if (M > 64 || K <= 0 || (K & 7) || (lda & 7) || (ldw & 7)) return IE_BAD_SIZE;
   if (((uintptr_t)A | (uintptr_t)W) & 15) return IE_BAD_ALIGN;
   if (nt != 1 && nt != 2 && nt != 4) return IE_BAD_SIZE;
-  if (epi == EPI_SILU_MUL && (N & 1)) return IE_BAD_SIZE;
+  if ((epi == EPI_SILU_MUL || epi == EPI_GLU) && (N & 1)) return IE_BAD_SIZE;
   StreamParams p;
   p.A = A; p.W = (const bf16*)W; p.C = C; p.gain = gain; p.row_index = row_index;
   p.M = M; p.N = N; p.K = K; p.lda = lda; p.ldw = ldw; p.ldc = ldc;
   p.gain_is_f32 = gain_dtype == IE_F32; p.eps = eps;
+  p.act_alpha = act_alpha; p.act_limit = act_limit; p.act_offset = act_offset; p.act_cubic = act_cubic;
   if (pro == PRO_NORM) {
     if (!gain || ((uintptr_t)gain & 15)) return IE_BAD_ALIGN;
     if (epi == EPI_BF16) return dispatch<PRO_NORM, EPI_BF16>(p, nt, stream);
@@ -299,6 +324,8 @@ extern "C" int ie_gemm_stream(const void* A, const void* W, void* C, const void*
     if (epi == EPI_F32) return dispatch<PRO_PLAIN, EPI_F32>(p, nt, stream);
     if (epi == EPI_RESIDUAL) return dispatch<PRO_PLAIN, EPI_RESIDUAL>(p, nt, stream);
     if (epi == EPI_SILU_MUL) return dispatch<PRO_PLAIN, EPI_SILU_MUL>(p, nt, stream);
+    if (epi == EPI_RELU2) return dispatch<PRO_PLAIN, EPI_RELU2>(p, nt, stream);
+    if (epi == EPI_GLU) return dispatch<PRO_PLAIN, EPI_GLU>(p, nt, stream);
     return IE_BAD_DTYPE;
   }
   return IE_BAD_DTYPE;

@@ -36,7 +36,7 @@ namespace {
 // Epilogues: ...; RESIDUAL_NORMOUT is RESIDUAL that also prepares the next product's PRENORMED input: for the norm that
 // comes next it writes bfloat16(new residual * gain) and its block's sums of squares of the new residual rows.
 enum { PRO_PLAIN = 0, PRO_NORM = 1, PRO_PRENORMED = 2 };
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SILU_MUL = 3, EPI_RESIDUAL_NORMOUT = 4 };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SILU_MUL = 3, EPI_RESIDUAL_NORMOUT = 4, EPI_RELU2 = 5, EPI_GLU = 6 };
 constexpr int SSQ_SLOT = 16;         // floats per block in the sums-of-squares array (one per activation row)
 
 constexpr int CONSUMER_WARPS = 8;
@@ -100,7 +100,21 @@ struct TmaParams {
   float* ssq_out;         // [SSQ_SLOT rows][ssq_blocks] this block's sums of squares of the new residual rows
   const float* ssq_in;    // [SSQ_SLOT rows][ssq_blocks] the sums of the product ahead (PRENORMED)
   int ssq_blocks;
+  float act_alpha, act_limit, act_offset, act_cubic;   // GLU
 };
+
+// the gated activation of the GLU epilogue: g' sigmoid(alpha g' + cubic g'^3) (u' + offset), g' = min(g, limit) and u' = u
+// clamped to [-limit, limit]
+template <typename P>
+__device__ __forceinline__ float stream_glu(const P& p, float g, float u) {
+  g = fminf(g, p.act_limit);
+  u = fminf(fmaxf(u, -p.act_limit), p.act_limit) + p.act_offset;
+  return g / (1.f + expf(-g * fmaf(p.act_cubic * g, g, p.act_alpha))) * u;
+}
+__device__ __forceinline__ float stream_relu2(float v) {
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -458,7 +472,11 @@ __device__ __forceinline__ void finish_units(const TmaParams& p, const BlockCtx&
               v1 *= inv_rms[m];
             }
             const bool has1 = n + 1 < p.N;
-            if (EPI == EPI_BF16) {
+            if (EPI == EPI_RELU2) {
+              v0 = stream_relu2(v0);
+              v1 = stream_relu2(v1);
+            }
+            if (EPI == EPI_BF16 || EPI == EPI_RELU2) {
               bf16* c = (bf16*)p.C + (size_t)m * p.ldc + n;
               if (has1 && ((((uintptr_t)c) & 3) == 0)) *reinterpret_cast<uint32_t*>(c) = pack2(v0, v1);
               else { c[0] = __float2bfloat16_rn(v0); if (has1) c[1] = __float2bfloat16_rn(v1); }
@@ -482,6 +500,8 @@ __device__ __forceinline__ void finish_units(const TmaParams& p, const BlockCtx&
               bf16* xg = p.xg_out + (size_t)m * p.ld_xg + n;
               if (has1 && ((((uintptr_t)xg) & 3) == 0)) *reinterpret_cast<uint32_t*>(xg) = pack2(r0 * g0, r1 * g1);
               else { xg[0] = __float2bfloat16_rn(r0 * g0); if (has1) xg[1] = __float2bfloat16_rn(r1 * g1); }
+            } else if (EPI == EPI_GLU) {
+              ((bf16*)p.C)[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn(stream_glu(p, v0, v1));
             } else {
               const float sg = 1.f / (1.f + expf(-v0));
               ((bf16*)p.C)[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn((v0 * sg) * v1);
@@ -643,11 +663,12 @@ extern "C" int ie_gemm_stream_trace_read(unsigned long long* out, int max_launch
 extern "C" int ie_gemm_stream_tma(const void* A, const void* W, void* C, const void* gain, int gain_dtype,
                                   const int* row_index, int M, int N, int K, int lda, int ldw, int ldc, float eps,
                                   int pro, int epi, int n_sms, void* xg, int ld_xg, const void* gain_next,
-                                  int gain_next_dtype, float* ssq, int ssq_blocks, cudaStream_t stream) {
+                                  int gain_next_dtype, float* ssq, int ssq_blocks, float act_alpha, float act_limit,
+                                  float act_offset, float act_cubic, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return IE_OK;
   if (!ie_gemm_stream_tma_supports(M, N, K, pro) || (lda & 7) || (ldw & 7)) return IE_BAD_SIZE;
   if (((uintptr_t)A | (uintptr_t)W) & 15) return IE_BAD_ALIGN;
-  if (epi == EPI_SILU_MUL && (N & 1)) return IE_BAD_SIZE;
+  if ((epi == EPI_SILU_MUL || epi == EPI_GLU) && (N & 1)) return IE_BAD_SIZE;
   if (n_sms <= 0) return IE_BAD_SIZE;
   TmaParams p;
   p.A = A; p.W = (const bf16*)W; p.C = C; p.gain = gain; p.row_index = row_index;
@@ -655,6 +676,7 @@ extern "C" int ie_gemm_stream_tma(const void* A, const void* W, void* C, const v
   p.gain_is_f32 = gain_dtype == IE_F32; p.eps = eps;
   p.xg_out = (bf16*)xg; p.ld_xg = ld_xg; p.gain_next = gain_next; p.gain_next_is_f32 = gain_next_dtype == IE_F32;
   p.ssq_out = ssq; p.ssq_in = ssq; p.ssq_blocks = ssq_blocks;
+  p.act_alpha = act_alpha; p.act_limit = act_limit; p.act_offset = act_offset; p.act_cubic = act_cubic;
   if (epi == EPI_RESIDUAL_NORMOUT &&
       (!xg || !gain_next || !ssq || ssq_blocks < n_sms || (ld_xg & 1) || (((uintptr_t)xg | (uintptr_t)ssq) & 3)))
     return IE_BAD_SIZE;
@@ -716,6 +738,8 @@ extern "C" int ie_gemm_stream_tma(const void* A, const void* W, void* C, const v
     if (epi == EPI_F32) return launch_tma<PRO_PLAIN, EPI_F32>(p, nt, n_sms, smem, stream);
     if (epi == EPI_RESIDUAL) return launch_tma<PRO_PLAIN, EPI_RESIDUAL>(p, nt, n_sms, smem, stream);
     if (epi == EPI_SILU_MUL) return launch_tma<PRO_PLAIN, EPI_SILU_MUL>(p, nt, n_sms, smem, stream);
+    if (epi == EPI_RELU2) return launch_tma<PRO_PLAIN, EPI_RELU2>(p, nt, n_sms, smem, stream);
+    if (epi == EPI_GLU) return launch_tma<PRO_PLAIN, EPI_GLU>(p, nt, n_sms, smem, stream);
     return IE_BAD_DTYPE;
   }
   return IE_BAD_DTYPE;

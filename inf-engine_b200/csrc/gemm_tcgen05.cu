@@ -5,6 +5,7 @@
 //   STORE_BF16   C bf16
 //   SILU_MUL     weight rows alternate gate_j, up_j; C[M, N/2] = silu(gate_j) * up_j   (engine/llama_mlp.py:30-32)
 //   RESIDUAL     C float32 [M, N] += product                                            (engine/llama_block.py:54,62)
+//   RELU2        C bf16, max(product, 0)^2: the first product of a feed-forward without a gate
 // The plain product is what the reference leaves to a library; the fused epilogues save the round trip of
 // the [M, 2*intermediate] gate/up matrix and of the projections' outputs through HBM.
 //
@@ -19,7 +20,7 @@
 
 namespace {
 
-enum { TC_EPI_BF16 = 0, TC_EPI_SILU_MUL = 3, TC_EPI_RESIDUAL = 2 };
+enum { TC_EPI_BF16 = 0, TC_EPI_SILU_MUL = 3, TC_EPI_RESIDUAL = 2, TC_EPI_RELU2 = 5 };
 
 constexpr int BM = 128;
 constexpr int BK = 64;               // one 128-byte swizzle atom of bfloat16
@@ -38,9 +39,10 @@ struct TcParams {
   int epi;
   int n_stages;
   int staged;   // the output's base and row pitch are multiples of 16 bytes: full tiles leave through shared memory
-  // SILU_MUL with options: g' = min(g, act_limit), u' = clamp(u, -act_limit, act_limit); g' sigmoid(act_alpha g') (u' + up_offset)
+  // SILU_MUL with options: g' = min(g, act_limit), u' = clamp(u, -act_limit, act_limit);
+  // g' sigmoid(act_alpha g' + act_cubic g'^3) (u' + up_offset)
   int act_general;
-  float act_alpha, act_limit, up_offset;
+  float act_alpha, act_limit, up_offset, act_cubic;
 };
 
 // the gated activation of the SILU_MUL epilogue: silu(g) * u, or with the options above
@@ -48,7 +50,15 @@ __device__ __forceinline__ float tc_glu(const TcParams& p, float g, float u) {
   if (!p.act_general) return __fdividef(g, 1.f + __expf(-g)) * u;
   g = fminf(g, p.act_limit);
   u = fminf(fmaxf(u, -p.act_limit), p.act_limit);
-  return __fdividef(g, 1.f + __expf(-p.act_alpha * g)) * (u + p.up_offset);
+  return __fdividef(g, 1.f + __expf(-g * fmaf(p.act_cubic * g, g, p.act_alpha))) * (u + p.up_offset);
+}
+
+// an accumulator as it is, or the square of its positive part
+__device__ __forceinline__ float tc_relu2(bool sq, uint32_t bits) {
+  const float v = __uint_as_float(bits);
+  if (!sq) return v;
+  const float r = fmaxf(v, 0.f);
+  return r * r;
 }
 
 __device__ __forceinline__ uint32_t saddr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -106,7 +116,8 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
 // one row's 32 accumulator columns n .. n+31 through the epilogue p.epi
 __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, int m, int n, const uint32_t (&r)[32]) {
   if (m < p.M && n < p.N) {
-    if (p.epi == TC_EPI_BF16) {
+    if (p.epi == TC_EPI_BF16 || p.epi == TC_EPI_RELU2) {
+      const bool sq = p.epi == TC_EPI_RELU2;
       bf16* dst = (bf16*)p.C + (size_t)m * p.ldc + n;
       if (n + 32 <= p.N && (((uintptr_t)dst) & 15) == 0) {
 #pragma unroll
@@ -115,13 +126,13 @@ __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, int m, int 
           __nv_bfloat162* vp = reinterpret_cast<__nv_bfloat162*>(&v);
 #pragma unroll
           for (int q = 0; q < 4; ++q)
-            vp[q] = __floats2bfloat162_rn(__uint_as_float(r[j * 8 + 2 * q]), __uint_as_float(r[j * 8 + 2 * q + 1]));
+            vp[q] = __floats2bfloat162_rn(tc_relu2(sq, r[j * 8 + 2 * q]), tc_relu2(sq, r[j * 8 + 2 * q + 1]));
           *reinterpret_cast<uint4*>(dst + j * 8) = v;
         }
       } else {
 #pragma unroll
         for (int j = 0; j < 32; ++j)
-          if (n + j < p.N) dst[j] = __float2bfloat16_rn(__uint_as_float(r[j]));
+          if (n + j < p.N) dst[j] = __float2bfloat16_rn(tc_relu2(sq, r[j]));
       }
     } else if (p.epi == TC_EPI_SILU_MUL) {
       bf16* dst = (bf16*)p.C + (size_t)m * p.ldc + (n >> 1);
@@ -175,20 +186,21 @@ __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, int m, int 
 constexpr int TC_STAGE_BYTES = 32 * 128;      // per epilogue warp
 
 // bytes of output that 32 accumulator columns make
-__device__ __forceinline__ int tc_out_bytes32(int epi) { return epi == TC_EPI_BF16 ? 64 : (epi == TC_EPI_SILU_MUL ? 32 : 128); }
+__device__ __forceinline__ int tc_out_bytes32(int epi) { return (epi == TC_EPI_BF16 || epi == TC_EPI_RELU2) ? 64 : (epi == TC_EPI_SILU_MUL ? 32 : 128); }
 
 // this lane's 32 accumulator columns -> its row of the warp's tile, from byte offset off
 __device__ __forceinline__ void tc_stage_row(const TcParams& p, unsigned char* stage, int lane, int off, int epi, const uint32_t (&r)[32]) {
   unsigned char* row = stage + lane * 128;
   const int u0 = off >> 4, sw = lane & 7;
-  if (epi == TC_EPI_BF16) {
+  if (epi == TC_EPI_BF16 || epi == TC_EPI_RELU2) {
+    const bool sq = epi == TC_EPI_RELU2;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       uint4 v;
       __nv_bfloat162* vp = reinterpret_cast<__nv_bfloat162*>(&v);
 #pragma unroll
       for (int q = 0; q < 4; ++q)
-        vp[q] = __floats2bfloat162_rn(__uint_as_float(r[j * 8 + 2 * q]), __uint_as_float(r[j * 8 + 2 * q + 1]));
+        vp[q] = __floats2bfloat162_rn(tc_relu2(sq, r[j * 8 + 2 * q]), tc_relu2(sq, r[j * 8 + 2 * q + 1]));
       *reinterpret_cast<uint4*>(row + (((u0 + j) ^ sw) << 4)) = v;
     }
   } else if (epi == TC_EPI_SILU_MUL) {
@@ -445,17 +457,18 @@ extern "C" int ie_gemm_tcgen05_supports(int M, int N, int K, int lda, int ldw) {
 }
 
 // epi: 0 bf16 out [M,N]; 2 float32 C[M,N] += product; 3 silu(gate)*up over interleaved weight rows, bf16 out [M, N/2]
+//      5 the square of max(product, 0), bf16 out [M,N]
 // bn:  tile width, 128 or 256
 // act_general != 0: the SILU_MUL epilogue clamps the gate from above and the up branch to [-act_limit, act_limit], scales
-// the sigmoid's argument by act_alpha and adds up_offset to the up branch
+// the sigmoid's argument by act_alpha, adds act_cubic times the gate's third power to it, and up_offset to the up branch
 extern "C" int ie_gemm_tcgen05_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,
                                    int epi, int bn, int n_sms, int act_general, float act_alpha, float act_limit,
-                                   float up_offset, cudaStream_t stream) {
+                                   float up_offset, float act_cubic, cudaStream_t stream) {
   if (n_sms <= 0) return IE_BAD_SIZE;
   if (M <= 0 || N <= 0) return IE_OK;
   if (!ie_gemm_tcgen05_supports(M, N, K, lda, ldw)) return IE_BAD_SIZE;
   if (((uintptr_t)A | (uintptr_t)W) & 15) return IE_BAD_ALIGN;
-  if (epi != TC_EPI_BF16 && epi != TC_EPI_SILU_MUL && epi != TC_EPI_RESIDUAL) return IE_BAD_DTYPE;
+  if (epi != TC_EPI_BF16 && epi != TC_EPI_SILU_MUL && epi != TC_EPI_RESIDUAL && epi != TC_EPI_RELU2) return IE_BAD_DTYPE;
   if (epi == TC_EPI_SILU_MUL && (N & 1)) return IE_BAD_SIZE;
   if (bn != 128 && bn != 256) return IE_BAD_SIZE;
   CUtensorMap ma, mw;
@@ -466,11 +479,12 @@ extern "C" int ie_gemm_tcgen05_act(const void* A, const void* W, void* C, int M,
   TcParams p;
   p.C = C; p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.epi = epi; p.n_stages = 0;
   p.act_general = act_general; p.act_alpha = act_alpha; p.act_limit = act_limit; p.up_offset = up_offset;
+  p.act_cubic = act_cubic;
   p.staged = (((uintptr_t)C & 15) == 0 && ((size_t)ldc * (epi == TC_EPI_RESIDUAL ? 4 : 2)) % 16 == 0) ? 1 : 0;
   return bn == 256 ? launch_tc<256>(ma, mw, p, n_sms, stream) : launch_tc<128>(ma, mw, p, n_sms, stream);
 }
 
 extern "C" int ie_gemm_tcgen05(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,
                                int epi, int bn, int n_sms, cudaStream_t stream) {
-  return ie_gemm_tcgen05_act(A, W, C, M, N, K, lda, ldw, ldc, epi, bn, n_sms, 0, 1.f, 0.f, 0.f, stream);
+  return ie_gemm_tcgen05_act(A, W, C, M, N, K, lda, ldw, ldc, epi, bn, n_sms, 0, 1.f, 0.f, 0.f, 0.f, stream);
 }

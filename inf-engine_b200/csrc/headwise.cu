@@ -1,6 +1,7 @@
 // Work on the heads of a token's projections, before and after attention.
 //
 // head_prepare: for every token, on the query side and on the key side, each with its own head count and head size:
+//   * an optional bias, one number a coordinate of the projection;
 //   * an optional RMS norm over the FIRST `norm_dims` dimensions of every head (x / sqrt(mean(x^2) + eps) * gain, gain of
 //     that size, shared by the heads; the other dimensions pass unchanged): a norm of whole heads when norm_dims is the
 //     head size, a norm of the compressed part of a key row that also carries a rotated part when it is less;
@@ -10,8 +11,11 @@
 //     inv_freq is float64 (blended frequencies of a scaled rotation are worked out on the host), the product with the
 //     position is formed and brought into one turn in double, sine and cosine are float32;
 //   * queries are written back in place, keys go to their page slot in a pool [page, key heads, page_size, head size]
-//     and values (optional, copied as they are) to [page, value heads, page_size, value size].
-// A token whose slot is negative (padding) writes nothing to the pools.
+//     and values (optional) to [page, value heads, page_size, value size]: rows of their own, copied as they are, or the
+//     keys with their bias before norm and rotation (`tied`: the layer has no projection of its own for them).
+// A token whose slot is negative (padding) writes nothing to the pools.  `rotate_write_kernel` is the form for bfloat16 rows
+// without norms, rotated in halves: eight coordinates (a rotated one with its partner's eight) a thread, the sines and
+// cosines of a block's tokens worked out once and shared by all heads.
 //
 // heads_gemm: a product per head, out[m, h, j] = sum_k x[m, h, k] * w[h, k, j], float32 products summed in ascending k
 // (the same for a row whatever else is in the batch), any of float32 and bfloat16 for x, w and out.
@@ -24,6 +28,7 @@ struct HeadSide {
   void* x;            // [n, heads * hd] rows, row stride `stride`
   int stride, heads, hd, norm_dims, rot_off;
   const void* gain;   // [norm_dims] or null
+  const void* bias;   // [heads * hd] or null, of the gains' type
 };
 
 template <typename TA, typename TW>
@@ -31,7 +36,7 @@ __global__ void head_prepare_kernel(HeadSide qs_, HeadSide ks_, const TA* __rest
                                     const double* __restrict__ inv_freq, int rot_dims, int neighbours, float mult,
                                     const int* __restrict__ positions, const int* __restrict__ slot_mapping,
                                     TA* __restrict__ kpool, TA* __restrict__ vpool, int n_v_heads, int hd_v,
-                                    int page_size) {
+                                    int page_size, int tied) {
   extern __shared__ float rows[];
   pdl_trigger();
   pdl_wait();
@@ -42,8 +47,18 @@ __global__ void head_prepare_kernel(HeadSide qs_, HeadSide ks_, const TA* __rest
   float* sk = rows + qw;
   TA* qr = (TA*)qs_.x + (size_t)n * qs_.stride;
   TA* kr = (TA*)ks_.x + (size_t)n * ks_.stride;
-  for (int i = threadIdx.x; i < qw; i += blockDim.x) sq[i] = to_f32(qr[i]);
-  for (int i = threadIdx.x; i < kw; i += blockDim.x) sk[i] = to_f32(kr[i]);
+  const int slot = slot_mapping ? IE_SLOT(slot_mapping[n]) : -1;
+  const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
+  for (int i = threadIdx.x; i < qw; i += blockDim.x)
+    sq[i] = to_f32(qr[i]) + (qs_.bias != nullptr ? to_f32(((const TW*)qs_.bias)[i]) : 0.f);
+  for (int i = threadIdx.x; i < kw; i += blockDim.x) {
+    const float x = to_f32(kr[i]) + (ks_.bias != nullptr ? to_f32(((const TW*)ks_.bias)[i]) : 0.f);
+    sk[i] = x;
+    if (tied && slot >= 0 && vpool != nullptr) {
+      const int h = i / ks_.hd, le = i - h * ks_.hd;
+      vpool[(((size_t)page * ks_.heads + h) * page_size + off) * ks_.hd + le] = from_f32<TA>(x);
+    }
+  }
   __syncthreads();
   // norms: a warp a head
   for (int side = 0; side < 2; ++side) {
@@ -62,8 +77,6 @@ __global__ void head_prepare_kernel(HeadSide qs_, HeadSide ks_, const TA* __rest
   }
   __syncthreads();
   const double pos = (double)positions[n];
-  const int slot = slot_mapping ? IE_SLOT(slot_mapping[n]) : -1;
-  const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
   const int half = rot_dims >> 1;
   for (int i = threadIdx.x; i < qw + kw; i += blockDim.x) {
     const bool is_q = i < qw;
@@ -105,10 +118,109 @@ __global__ void head_prepare_kernel(HeadSide qs_, HeadSide ks_, const TA* __rest
   }
 }
 
+#define RW_THREADS 256
+
+struct RotateWriteParams {
+  bf16* q;
+  const bf16* k;
+  const void* q_bias;
+  const void* k_bias;
+  int q_stride, k_stride, q_heads, k_heads, hd, rot_dims, page_size, tied, n_tokens, tokens_a_block;
+  const double* inv_freq;
+  float mult;
+  const int* positions;
+  const int* slot_mapping;
+  bf16* kpool;
+  bf16* vpool;
+};
+
+template <typename TW>
+__device__ __forceinline__ void load8_biased(const bf16* x, const TW* bias, float (&f)[8]) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(x);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 v = __bfloat1622float2(h[i]);
+    f[2 * i] = v.x;
+    f[2 * i + 1] = v.y;
+  }
+  if (bias == nullptr) return;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) f[i] += to_f32(bias[i]);
+}
+__device__ __forceinline__ void store8(bf16* dst, const float (&f)[8]) {
+  uint4 raw;
+  __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+  *reinterpret_cast<uint4*>(dst) = raw;
+}
+
+template <typename TW>
+__global__ void __launch_bounds__(RW_THREADS) rotate_write_kernel(RotateWriteParams p) {
+  extern __shared__ float2 cs_sn[];                       // [tokens_a_block][rot_dims / 2]
+  pdl_trigger();
+  pdl_wait();
+  const int t0 = blockIdx.x * p.tokens_a_block, nt = min(p.tokens_a_block, p.n_tokens - t0);
+  const int half = p.rot_dims >> 1;
+  for (int i = threadIdx.x; i < nt * half; i += RW_THREADS) {
+    const int t = i / half, pair = i - t * half;
+    const double turns = (double)p.positions[t0 + t] * p.inv_freq[pair] * 0.15915494309189535;
+    float2 v;
+    sincosf((float)((turns - floor(turns)) * 6.283185307179586), &v.y, &v.x);
+    cs_sn[i] = make_float2(v.x * p.mult, v.y * p.mult);
+  }
+  __syncthreads();
+  const int pair_units = p.rot_dims >> 4, units = pair_units + ((p.hd - p.rot_dims) >> 3);
+  const int per_token = (p.q_heads + p.k_heads) * units;
+  for (int it = threadIdx.x; it < nt * per_token; it += RW_THREADS) {
+    const int t = it / per_token, r = it - t * per_token;
+    const int head = r / units, u = r - head * units;
+    const bool is_q = head < p.q_heads;
+    const int h = is_q ? head : head - p.q_heads;
+    const bool turned = u < pair_units;
+    const int d = turned ? u * 8 : p.rot_dims + (u - pair_units) * 8;
+    const size_t n = t0 + t;
+    const bf16* src = (is_q ? p.q + n * p.q_stride : p.k + n * p.k_stride) + h * p.hd + d;
+    const TW* bias = (const TW*)(is_q ? p.q_bias : p.k_bias);
+    if (bias != nullptr) bias += h * p.hd + d;
+    bf16 *dst = const_cast<bf16*>(src), *vdst = nullptr;
+    if (!is_q) {
+      const int slot = p.slot_mapping != nullptr ? IE_SLOT(p.slot_mapping[n]) : -1;
+      if (slot < 0 || p.kpool == nullptr) continue;
+      const size_t at = (((size_t)(slot / p.page_size) * p.k_heads + h) * p.page_size + slot % p.page_size) * p.hd + d;
+      dst = p.kpool + at;
+      if (p.tied && p.vpool != nullptr) vdst = p.vpool + at;
+    }
+    float a[8];
+    load8_biased<TW>(src, bias, a);
+    if (vdst != nullptr) store8(vdst, a);
+    if (!turned) {
+      store8(dst, a);
+      continue;
+    }
+    float b[8];
+    load8_biased<TW>(src + half, bias != nullptr ? bias + half : nullptr, b);
+    if (vdst != nullptr) store8(vdst + half, b);
+    const float2* cs = cs_sn + t * half + d;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float2 c = cs[i];
+      const float x = a[i], y = b[i];
+      a[i] = fmaf(x, c.x, -y * c.y);
+      b[i] = fmaf(y, c.x, x * c.y);
+    }
+    store8(dst, a);
+    store8(dst + half, b);
+  }
+}
+
+// tied: the key rows with their bias, before norm and rotation, are also the values (v is then ignored; the pool has the
+// keys' heads and head size)
 extern "C" int ie_head_prepare(void* q, int q_stride, int q_heads, int q_hd, int q_norm_dims, int q_rot_off,
                                const void* q_gain, void* k, int k_stride, int k_heads, int k_hd, int k_norm_dims,
-                               int k_rot_off, const void* k_gain, int w_dtype, const void* v, int v_stride,
-                               int n_v_heads, int hd_v, float eps, const double* inv_freq, int rot_dims, int neighbours,
+                               int k_rot_off, const void* k_gain, const void* q_bias, const void* k_bias, int w_dtype,
+                               const void* v, int v_stride, int tied, int n_v_heads, int hd_v, float eps, const double* inv_freq, int rot_dims, int neighbours,
                                float mult, const int* positions, const int* slot_mapping, void* kpool, void* vpool,
                                int n_tokens, int page_size, int act_dtype, cudaStream_t stream) {
   if (n_tokens <= 0) return IE_OK;
@@ -117,8 +229,25 @@ extern "C" int ie_head_prepare(void* q, int q_stride, int q_heads, int q_hd, int
   if (inv_freq != nullptr && (q_rot_off < 0 || k_rot_off < 0 || q_rot_off + rot_dims > q_hd || k_rot_off + rot_dims > k_hd))
     return IE_BAD_SIZE;
   if (q_norm_dims > q_hd || k_norm_dims > k_hd) return IE_BAD_SIZE;
-  HeadSide qs{q, q_stride, q_heads, q_hd, q_norm_dims, q_rot_off, q_gain};
-  HeadSide ks{k, k_stride, k_heads, k_hd, k_norm_dims, k_rot_off, k_gain};
+  HeadSide qs{q, q_stride, q_heads, q_hd, q_norm_dims, q_rot_off, q_gain, q_bias};
+  HeadSide ks{k, k_stride, k_heads, k_hd, k_norm_dims, k_rot_off, k_gain, k_bias};
+  if (tied) v = nullptr;
+  const uintptr_t at = (uintptr_t)q | (uintptr_t)k | (uintptr_t)q_bias | (uintptr_t)k_bias | (uintptr_t)kpool | (uintptr_t)vpool;
+  const int rot = inv_freq != nullptr ? rot_dims : 0;
+  if (act_dtype == IE_BF16 && q_gain == nullptr && k_gain == nullptr && v == nullptr && !neighbours && q_rot_off == 0 &&
+      k_rot_off == 0 && q_hd == k_hd && q_hd % 8 == 0 && rot % 16 == 0 && q_stride % 8 == 0 && k_stride % 8 == 0 && (at & 15) == 0 &&
+      q_heads + k_heads > 0) {
+    RotateWriteParams p;
+    p.q = (bf16*)q; p.k = (const bf16*)k; p.q_bias = q_bias; p.k_bias = k_bias; p.q_stride = q_stride; p.k_stride = k_stride;
+    p.q_heads = q_heads; p.k_heads = k_heads; p.hd = q_hd; p.rot_dims = rot; p.page_size = page_size; p.tied = tied;
+    p.n_tokens = n_tokens; p.tokens_a_block = n_tokens >= 1024 ? 4 : (n_tokens >= 512 ? 2 : 1); p.inv_freq = inv_freq;
+    p.mult = mult; p.positions = positions; p.slot_mapping = slot_mapping; p.kpool = (bf16*)kpool; p.vpool = (bf16*)vpool;
+    const int blocks = (n_tokens + p.tokens_a_block - 1) / p.tokens_a_block;
+    const size_t cs_bytes = sizeof(float2) * p.tokens_a_block * (size_t)(rot >> 1);
+    if (w_dtype == IE_F32) return launch_k(rotate_write_kernel<float>, blocks, RW_THREADS, cs_bytes, stream, p);
+    if (w_dtype == IE_BF16) return launch_k(rotate_write_kernel<bf16>, blocks, RW_THREADS, cs_bytes, stream, p);
+    return IE_BAD_DTYPE;
+  }
   const size_t smem = sizeof(float) * ((size_t)q_heads * q_hd + (size_t)k_heads * k_hd);
   if (smem > 200 * 1024) return IE_BAD_SIZE;
   const int threads = 256;
@@ -131,7 +260,7 @@ extern "C" int ie_head_prepare(void* q, int q_stride, int q_heads, int q_hd, int
     }                                                                                                              \
     return launch_k(head_prepare_kernel<TA, TW>, n_tokens, threads, smem, stream, qs, ks, (const TA*)v, v_stride,  \
                     eps, inv_freq, rot_dims, neighbours, mult, positions, slot_mapping, (TA*)kpool, (TA*)vpool,    \
-                    n_v_heads, hd_v, page_size);                                                                   \
+                    n_v_heads, hd_v, page_size, tied);                                                                   \
   }
   if (act_dtype == IE_F32 && w_dtype == IE_F32) HP_GO(float, float);
   if (act_dtype == IE_F32 && w_dtype == IE_BF16) HP_GO(float, bf16);

@@ -5,8 +5,8 @@
 //            (mode 2) as mode 0 with the softmax over all experts as the scores.  A group's score is the sum of its two
 //            largest choice scores or (group_max) the largest one;
 //   sort     the (token, choice) pairs ordered by expert, and a table of row tiles, none of which spans two experts;
-//   product  C[pair] = A[token of pair] W[expert of pair]^T over those tiles, optionally with the gated activation in the
-//            epilogue: on CUDA cores (float32 products and sums, every output one accumulator that walks k upward) for
+//   product  C[pair] = A[token of pair] W[expert of pair]^T over those tiles, optionally with the gated activation, or the
+//            square of relu of an expert without a gate, in the epilogue: on CUDA cores (float32 products and sums, every output one accumulator that walks k upward) for
 //            the 32-bit path, on tensor cores (mma.sync, float32 accumulators) for bfloat16 operands; either way a
 //            row's result does not depend on which tile or step it is in;
 //   combine  out[token] = sum over its choices of weight * y[pair] + gate * shared[token], choices in order.
@@ -190,15 +190,21 @@ extern "C" int ie_moe_sort(const int* ids, int n_pairs, int n_experts, int tile_
 }
 
 // ------------------------------------------------------------------ grouped product
-// The activation of a gated expert: g' sigmoid(alpha g') * (u' + up_offset), g' = min(g, limit) and u' = u clamped to
-// [-limit, limit] (silu(g) * u: alpha 1, an infinite limit, no offset).
+// The activation of a gated expert: g' sigmoid(alpha g' + cubic g'^3) * (u' + up_offset), g' = min(g, limit) and u' = u
+// clamped to [-limit, limit] (silu(g) * u: alpha 1, an infinite limit, no offset, no third power).
 struct GluAct {
-  float alpha, limit, up_offset;
+  float alpha, limit, up_offset, cubic;
 };
+// what an epilogue without a gate stores: the sum as it is, or (epi 2) the square of its positive part
+__device__ __forceinline__ float plain_act(int epi, float v) {
+  if (epi != 2) return v;
+  const float r = fmaxf(v, 0.f);
+  return r * r;
+}
 __device__ __forceinline__ float glu(const GluAct& a, float g, float u) {
   g = fminf(g, a.limit);
   u = fminf(fmaxf(u, -a.limit), a.limit) + a.up_offset;
-  return g / (1.f + expf(-a.alpha * g)) * u;
+  return g / (1.f + expf(-g * fmaf(a.cubic * g, g, a.alpha))) * u;
 }
 
 #define MG_BM 64
@@ -209,7 +215,7 @@ __device__ __forceinline__ float glu(const GluAct& a, float g, float u) {
 // A row of tile (expert e, positions pos0 .. pos0 + rows): gather = 1: row sorted[pos] / top of A (a token's
 // activations); gather = 0: row pos of A (what the product before left in sorted order).  C row: scatter = 1: row
 // sorted[pos] (the pair's own place), else row pos.  W is [experts, N, K].  epi 1: columns alternate gate, up and the
-// output is the gated activation, N / 2 wide.
+// output is the gated activation, N / 2 wide; epi 2: the square of the sum's positive part, N wide.
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(MG_THREADS)
 moe_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restrict__ C, const int* __restrict__ sorted,
@@ -285,7 +291,7 @@ moe_gemm_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restri
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int n = n0 + tx * 4 + j;
-        if (n < N) C[(size_t)cr * ldc + n] = from_f32<TC>(acc[i][j]);
+        if (n < N) C[(size_t)cr * ldc + n] = from_f32<TC>(plain_act(epi, acc[i][j]));
       }
     }
   }
@@ -415,8 +421,8 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* 
         if (epi == 1) {
           if (n + 1 < N) C[(size_t)cr * ldc + (n >> 1)] = from_f32<TC>(glu(act, x0, x1));
         } else {
-          if (n < N) C[(size_t)cr * ldc + n] = from_f32<TC>(x0);
-          if (n + 1 < N) C[(size_t)cr * ldc + n + 1] = from_f32<TC>(x1);
+          if (n < N) C[(size_t)cr * ldc + n] = from_f32<TC>(plain_act(epi, x0));
+          if (n + 1 < N) C[(size_t)cr * ldc + n + 1] = from_f32<TC>(plain_act(epi, x1));
         }
       }
     }
@@ -428,8 +434,8 @@ extern "C" int ie_moe_tile_rows() { return MG_BM; }
 extern "C" int ie_moe_gemm(const void* A, int a_dtype, const void* W, int w_dtype, void* C, int c_dtype,
                            const int* sorted, const int* tiles, int max_tiles, int N, int K, int lda, int ldc,
                            long long w_expert_stride, int top, int gather, int scatter, int epi, float alpha, float limit,
-                           float up_offset, cudaStream_t stream) {
-  const GluAct act{alpha, limit, up_offset};
+                           float up_offset, float cubic, cudaStream_t stream) {
+  const GluAct act{alpha, limit, up_offset, cubic};
   if (max_tiles <= 0 || N <= 0) return IE_OK;
   if (K <= 0 || top <= 0 || (epi == 1 && (N & 1))) return IE_BAD_SIZE;
   if (a_dtype == IE_BF16 && w_dtype == IE_BF16 && K % 8 == 0 && lda % 8 == 0 && w_expert_stride % 8 == 0 &&

@@ -100,15 +100,17 @@ def core():
         lib.ie_rownorm_rotate_write.argtypes = [P, P, P, I, I, I, P, P, P, P, P, I, F, P, I, P, P, P, P, I, I, I, I, I, I, I, P]
         lib.ie_moe_route.argtypes = [P, I, P, I, P, P, P, I, I, I, I, I, F, F, I, I, I, P]
         lib.ie_moe_sort.argtypes = [P, I, I, I, P, P, I, P]
-        lib.ie_moe_gemm.argtypes = [P, I, P, I, P, I, P, P, I, I, I, I, I, L, I, I, I, I, F, F, F, P]
+        lib.ie_moe_gemm.argtypes = [P, I, P, I, P, I, P, P, I, I, I, I, I, L, I, I, I, I, F, F, F, F, P]
         lib.ie_moe_combine.argtypes = [P, P, P, P, I, I, P, I, I, I, P]
         lib.ie_moe_tile_rows.restype = c_int
-        lib.ie_head_prepare.argtypes = [P, I, I, I, I, I, P, P, I, I, I, I, I, P, I, P, I, I, I, F, P, I, I, F, P, P, P, P, I, I, I, P]
+        lib.ie_head_prepare.argtypes = [P, I, I, I, I, I, P, P, I, I, I, I, I, P, P, P, I, P, I, I, I, I, F, P, I, I, F, P, P, P, P, I, I, I, P]
         lib.ie_heads_gemm.argtypes = [P, I, I, I, P, I, P, I, I, I, I, I, I, I, P]
         lib.ie_diff_combine.argtypes = [P, I, P, I, P, I, I, I, I, I, F, F, F, I, P]
         lib.ie_gated_residual_add.argtypes = [P, P, I, P, I, P, I, I, I, I, P]
         lib.ie_scale_rows.argtypes = [P, P, F, I, I, P]
-        lib.ie_glu_act.argtypes = [P, P, I, I, I, I, I, F, F, F, I, P]
+        lib.ie_glu_act.argtypes = [P, P, I, I, I, I, I, F, F, F, F, I, P]
+        lib.ie_relu2.argtypes = [P, I, P, I, I, I, I, P]
+        lib.ie_softcap.argtypes = [P, F, ctypes.c_size_t, P]
         lib.ie_mingru_scan.argtypes = [P, P, I, P, I, P, P, I, P, P, I, P, P, I, I, I, I, P]
         lib.ie_mingru_scan_hint.argtypes = [P, P, I, P, I, P, P, I, P, P, I, P, P, I, I, I, I, I, P]
         D = ctypes.c_double
@@ -123,7 +125,7 @@ def core():
         lib.ie_mlstm_chunks.argtypes = [I, I]
         lib.ie_mlstm_state_floats.argtypes = [I, I]
         lib.ie_mlstm_state_floats.restype = c_longlong
-        lib.ie_stream_norm.argtypes = [P, P, I, I, P, P, I, P, I, I, F, P, I, P, I, I, P]
+        lib.ie_stream_norm.argtypes = [P, P, I, I, P, F, P, I, P, I, P, I, I, P, I, I, F, P, F, P, I, P, I, I, P]
         lib.ie_conv_qkv.argtypes = [P, I, P, P, L, I, I, P, I, P, P, P, I, F, P, I, I, F, P, P, P, P] + [I] * 11 + [P]
         lib.ie_argmax.argtypes = [P, P, I, I, L, P]
         lib.ie_repetition_penalty.argtypes = [P, P, P, I, I, L, I, P]
@@ -137,7 +139,7 @@ def core():
                      "ie_heads_gemm", "ie_diff_combine", "ie_gated_residual_add", "ie_scale_rows", "ie_glu_act",
                      "ie_mingru_scan", "ie_mingru_scan_hint", "ie_scale_add_sinusoid", "ie_add_row", "ie_token_shift",
                      "ie_gate_mul", "ie_qkv_prepare", "ie_talk_combine", "ie_mlstm_scan", "ie_mlstm_finish",
-                     "ie_mlstm_chunks", "ie_stream_norm", "ie_conv_qkv"):
+                     "ie_mlstm_chunks", "ie_stream_norm", "ie_conv_qkv", "ie_relu2", "ie_softcap"):
             getattr(lib, name).restype = c_int
         _core = lib
         _apply_check_limits()
@@ -496,25 +498,30 @@ def head_prepare(q: torch.Tensor, q_heads: int, q_head_dim: int, k: torch.Tensor
                  k_norm_dims: int = 0, eps: float = 0.0, inv_freq: torch.Tensor | None = None, rot_dims: int = 0,
                  q_rot_off: int = 0, k_rot_off: int = 0, neighbours: bool = False, mult: float = 1.0,
                  v: torch.Tensor | None = None, vpool: torch.Tensor | None = None, n_v_heads: int = 0,
-                 v_head_dim: int = 0) -> None:
-    """Per token: an RMS norm over the first ``*_norm_dims`` dimensions of every query head and key head (gains of that
+                 v_head_dim: int = 0, q_bias: torch.Tensor | None = None, k_bias: torch.Tensor | None = None,
+                 tied: bool = False) -> None:
+    """Per token: ``q_bias`` / ``k_bias`` ([heads * head_dim], optional) added; an RMS norm over the first ``*_norm_dims`` dimensions of every query head and key head (gains of that
     size; None: no norm), a rotation by position of ``rot_dims`` dimensions that start at ``*_rot_off`` of every head
     (``inv_freq`` float64 [rot_dims / 2]; in halves, or in neighbouring pairs with ``neighbours``; sine and cosine times
     ``mult``); q is written back in place, the keys go to their slots of ``kpool`` [pages, k_heads, page_size,
-    k_head_dim] and ``v`` (optional, as it is) to ``vpool`` [pages, n_v_heads, page_size, v_head_dim]."""
+    k_head_dim] and ``v`` (optional, as it is) to ``vpool`` [pages, n_v_heads, page_size, v_head_dim].  ``tied``: the keys
+    with their bias, before norm and rotation, are the values (``vpool`` has the shape of ``kpool``; no ``v``)."""
     n = q.shape[0]
     assert q.stride(1) == 1 and k.stride(1) == 1 and q.dtype == k.dtype and (v is None or (v.stride(1) == 1 and v.dtype == q.dtype))
-    gains = [g for g in (q_gain, k_gain) if g is not None]
+    gains = [g for g in (q_gain, k_gain, q_bias, k_bias) if g is not None]
     assert all(g.dtype == gains[0].dtype and g.is_contiguous() for g in gains)
+    assert q_bias is None or q_bias.numel() == q_heads * q_head_dim
+    assert k_bias is None or k_bias.numel() == k_heads * k_head_dim
+    assert not tied or (v is None and (vpool is None or (kpool is not None and vpool.shape == kpool.shape and vpool.dtype == kpool.dtype)))
     assert q_gain is None or q_gain.numel() >= q_norm_dims
     assert k_gain is None or k_gain.numel() >= k_norm_dims
     assert inv_freq is None or (inv_freq.dtype is torch.float64 and inv_freq.is_contiguous() and inv_freq.numel() * 2 >= rot_dims)
     assert kpool is None or kpool.dtype == q.dtype
     _check(core().ie_head_prepare(_ptr(q), q.stride(0), q_heads, q_head_dim, int(q_norm_dims if q_gain is not None else 0),
                                   int(q_rot_off), _ptr(q_gain), _ptr(k), k.stride(0), k_heads, k_head_dim,
-                                  int(k_norm_dims if k_gain is not None else 0), int(k_rot_off), _ptr(k_gain),
+                                  int(k_norm_dims if k_gain is not None else 0), int(k_rot_off), _ptr(k_gain), _ptr(q_bias), _ptr(k_bias),
                                   dtype_code(gains[0].dtype) if gains else IE_F32, _ptr(v),
-                                  v.stride(0) if v is not None else 0, int(n_v_heads), int(v_head_dim), float(eps),
+                                  v.stride(0) if v is not None else 0, 1 if tied else 0, int(n_v_heads), int(v_head_dim), float(eps),
                                   _ptr(inv_freq), int(rot_dims if inv_freq is not None else 0), 1 if neighbours else 0,
                                   float(mult), _ptr(positions), _ptr(slot_mapping), _ptr(kpool), _ptr(vpool), n,
                                   page_size, dtype_code(q.dtype), _stream()), "head_prepare")
@@ -565,19 +572,52 @@ def scale_rows(x: torch.Tensor, scale: float, keep: torch.Tensor | None = None) 
     _check(core().ie_scale_rows(_ptr(x), _ptr(keep), float(scale), x.shape[0], x.shape[1], _stream()), "scale_rows")
 
 
-GLU_KINDS = {"silu": 0, "clamped_swish": 1}
+GLU_KINDS = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 1}
+GELU_ALPHA = 2.0 * (2.0 / 3.141592653589793) ** 0.5     # the tanh form of gelu: g sigmoid(GELU_ALPHA (g + 0.044715 g^3))
+GELU_CUBIC = 0.044715 * GELU_ALPHA
+
+
+def glu_constants(kind: str, alpha: float = 1.0, limit: float = 0.0, up_offset: float = 0.0) -> tuple[float, float, float, float]:
+    """(alpha, limit, up_offset, cubic) of a gated activation, as the products' epilogues take it: ``g' sigmoid(alpha g' +
+    cubic g'^3) * (u' + up_offset)`` with g' = min(g, limit) and u' = u clamped to [-limit, limit]."""
+    if kind == "silu":
+        return 1.0, float("inf"), float(up_offset), 0.0
+    if kind == "clamped_swish":
+        return float(alpha), float(limit), float(up_offset), 0.0
+    if kind == "gelu_tanh":
+        return GELU_ALPHA, float("inf"), float(up_offset), GELU_CUBIC
+    raise KeyError(f"gated activation {kind!r} is not built (known: {sorted(GLU_KINDS)})")
+
+
+def _act4(act: tuple | None) -> tuple[float, float, float, float]:
+    """Activation constants of a product's epilogue: silu when none are given; the third power's is 0 unless named."""
+    return tuple(float(a) for a in (tuple(act) + (0.0,))[:4]) if act is not None else glu_constants("silu")
 
 
 def glu_act(gate_up: torch.Tensor, out: torch.Tensor, kind: str, interleaved: bool = False, alpha: float = 1.0,
             limit: float = 0.0, up_offset: float = 0.0) -> None:
     """out[n, j] = act(gate_j) * (up_j + up_offset).  ``silu``: g sigmoid(g).  ``clamped_swish``: g' sigmoid(alpha g')
-    with g' = min(g, limit), and up clamped to [-limit, limit].  Gate and up are the two halves of a row, or alternate
+    with g' = min(g, limit), and up clamped to [-limit, limit].  ``gelu_tanh``: the tanh form of gelu.  Gate and up are the two halves of a row, or alternate
     when ``interleaved``."""
     n, inter = out.shape
     assert gate_up.shape == (n, 2 * inter) and gate_up.stride(1) == 1 and out.is_contiguous() and gate_up.dtype == out.dtype
+    alpha, limit, up_offset, cubic = glu_constants(kind, alpha, limit, up_offset)
     _check(core().ie_glu_act(_ptr(gate_up), _ptr(out), n, inter, gate_up.stride(0), 1 if interleaved else 0,
-                             GLU_KINDS[kind], float(alpha), float(limit), float(up_offset), dtype_code(out.dtype),
-                             _stream()), f"glu_act({kind})")
+                             GLU_KINDS[kind], alpha, limit, up_offset, cubic, dtype_code(out.dtype), _stream()),
+           f"glu_act({kind})")
+
+
+def relu2(x: torch.Tensor, out: torch.Tensor) -> None:
+    """out = max(x, 0)^2, element by element (rows may have a stride; ``out`` may be ``x``)."""
+    n, cols = x.shape
+    assert out.shape == x.shape and out.dtype == x.dtype and x.stride(1) == 1 and out.stride(1) == 1
+    _check(core().ie_relu2(_ptr(x), x.stride(0), _ptr(out), out.stride(0), n, cols, dtype_code(x.dtype), _stream()), "relu2")
+
+
+def softcap(x: torch.Tensor, cap: float) -> None:
+    """x (float32, contiguous) <- cap * tanh(x / cap), in place."""
+    assert x.dtype is torch.float32 and x.is_contiguous() and cap > 0
+    _check(core().ie_softcap(_ptr(x), float(cap), x.numel(), _stream()), "softcap")
 
 
 def mingru_scan(z_pre: torch.Tensor, u_pre: torch.Tensor, g_pre: torch.Tensor, z_bias: torch.Tensor | None,
@@ -764,19 +804,18 @@ def moe_sort(ids: torch.Tensor, n_experts: int, sorted_pairs: torch.Tensor, tile
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, sorted_pairs: torch.Tensor, tiles: torch.Tensor,
-             top: int, gather: bool, scatter: bool, epi: str = "store", act: tuple[float, float, float] | None = None) -> None:
+             top: int, gather: bool, scatter: bool, epi: str = "store", act: tuple | None = None) -> None:
     """The grouped product over the tiles of ``moe_sort``: ``w`` [experts, N, K]; ``gather``: a pair's row of ``a`` is
     its token's (pair // top), else its sorted position; ``scatter``: its row of ``c`` is the pair's index, else its
     sorted position; ``epi`` "silu_mul": w's rows alternate gate, up and c, N / 2 wide, takes the gated activation: silu(g) *
-    u, or with ``act`` = (alpha, limit, up_offset) g' sigmoid(alpha g') * (u' + up_offset), g' = min(g, limit), u' = u
-    clamped to [-limit, limit]."""
-    alpha, limit, up_offset = act if act is not None else (1.0, float("inf"), 0.0)
+    u, or with ``act`` the activation of ``glu_constants``; ``epi`` "relu2": c takes max(product, 0)^2, N wide."""
+    alpha, limit, up_offset, cubic = _act4(act)
     _, n, k = w.shape
     assert w.is_contiguous() and a.stride(1) == 1 and c.stride(1) == 1 and a.shape[1] == k
     _check(core().ie_moe_gemm(_ptr(a), dtype_code(a.dtype), _ptr(w), dtype_code(w.dtype), _ptr(c), dtype_code(c.dtype),
                               _ptr(sorted_pairs), _ptr(tiles), tiles.shape[0], n, k, a.stride(0), c.stride(0), n * k, top,
-                              1 if gather else 0, 1 if scatter else 0, {"store": 0, "silu_mul": 1}[epi], float(alpha), float(limit),
-                              float(up_offset), _stream()),
+                              1 if gather else 0, 1 if scatter else 0, {"store": 0, "silu_mul": 1, "relu2": 2}[epi], float(alpha),
+                              float(limit), float(up_offset), float(cubic), _stream()),
            f"moe_gemm(n={n}, k={k}, {epi})")
 
 
@@ -796,13 +835,20 @@ def moe_combine(y: torch.Tensor, weights: torch.Tensor, gate: torch.Tensor | Non
 # ------------------------------------------------- a scaled sum into the stream, convolved queries, keys and values
 def stream_norm(residual: torch.Tensor, y: torch.Tensor | None, scale: torch.Tensor | None, weights: torch.Tensor | None,
                 gain: torch.Tensor | None, groups: int, eps: float, out: torch.Tensor | None,
-                row_index: torch.Tensor | None = None) -> None:
-    """residual (float32 [n, d]) += scale * y, coordinate by coordinate (``scale`` float32 [d], None: 1; ``y`` None:
-    nothing is added), and ``out`` (None: the sum alone) = the RMS norm of the new rows in ``groups`` equal consecutive
+                row_index: torch.Tensor | None = None, mult: float = 1.0, extras: tuple = (),
+                tanh: tuple[float, torch.Tensor] | None = None) -> None:
+    """residual (float32 [n, d]) += mult * scale * (y + sum of extras), coordinate by coordinate (``scale`` float32 [d],
+    None: 1; ``y`` None: nothing is added; ``extras``: up to two [n, d] summands of one type), and ``out`` (None: the sum alone) = the RMS norm of the new rows in ``groups`` equal consecutive
     parts, each by itself, times ``gain``.  With ``weights`` (float32 [n, top]) ``y`` is [n * top, d] and a row's summand
     is ``sum_r weights[n, r] * y[n * top + r]``.  With ``row_index`` only those rows are normed and the residual keeps
-    its values."""
+    its values.  ``tanh`` = (alpha, bias): ``out`` is tanh(alpha x) * gain + bias instead of the norm."""
     n, d = residual.shape
+    extras = tuple(e for e in extras if e is not None)
+    assert len(extras) <= 2 and (y is not None or not extras)
+    assert all(e.shape == (n, d) and e.stride(1) == 1 and e.dtype == extras[0].dtype for e in extras)
+    alpha, bias = tanh if tanh is not None else (0.0, None)
+    assert tanh is None or (out is not None and bias.shape == (d,) and bias.dtype == gain.dtype and bias.is_contiguous())
+    e0, e1 = (extras + (None, None))[:2]
     top = weights.shape[1] if weights is not None else 1
     assert residual.dtype is torch.float32 and residual.is_contiguous()
     assert y is None or (y.stride(1) == 1 and y.shape == (n * top, d))
@@ -811,8 +857,11 @@ def stream_norm(residual: torch.Tensor, y: torch.Tensor | None, scale: torch.Ten
     assert out is None or (out.is_contiguous() and out.shape[1] == d and gain.is_contiguous() and gain.shape == (d,))
     assert row_index is not None or out is None or out.shape[0] == n
     _check(core().ie_stream_norm(_ptr(residual), _ptr(y), dtype_code(y.dtype) if y is not None else IE_F32,
-                                 y.stride(0) if y is not None else d, _ptr(scale), _ptr(weights), top, _ptr(gain),
-                                 dtype_code(gain.dtype) if gain is not None else IE_F32, int(groups), float(eps), _ptr(out),
+                                 y.stride(0) if y is not None else d, _ptr(scale), float(mult), _ptr(weights), top,
+                                 _ptr(e0), e0.stride(0) if e0 is not None else 0, _ptr(e1),
+                                 e1.stride(0) if e1 is not None else 0, dtype_code(e0.dtype) if e0 is not None else IE_F32,
+                                 _ptr(gain), dtype_code(gain.dtype) if gain is not None else IE_F32, int(groups), float(eps),
+                                 _ptr(bias), float(alpha), _ptr(out),
                                  dtype_code(out.dtype) if out is not None else IE_F32, _ptr(row_index),
                                  out.shape[0] if out is not None else n, d, _stream()), f"stream_norm(groups={groups})")
 
@@ -1236,7 +1285,7 @@ def gated_delta(q, k, v, b_pre, a_pre, gate, a_log, dt_bias, out_gain, state, ou
 # ----------------------------------------------- weight-streaming product for few rows
 STREAM_MAX_ROWS = 64        # what the kernel takes
 STREAM_BEST_ROWS = 16       # beyond this the library product is faster (activations are re-read per block)
-_EPI = {"bf16": 0, "f32": 1, "residual": 2, "silu_mul": 3, "residual_normout": 4}
+_EPI = {"bf16": 0, "f32": 1, "residual": 2, "silu_mul": 3, "residual_normout": 4, "relu2": 5, "glu": 6}
 SSQ_SLOT = 16               # rows of a sums-of-squares array ([SSQ_SLOT, blocks]: a block's sum for each activation row)
 _stream_lib = None
 _stream_variants: dict = {}
@@ -1244,9 +1293,9 @@ _stream_variants: dict = {}
 
 def _bind_stream(lib):
     P, I, F = c_void_p, c_int, c_float
-    lib.ie_gemm_stream.argtypes = [P, P, P, P, I, P, I, I, I, I, I, I, F, I, I, I, P]
+    lib.ie_gemm_stream.argtypes = [P, P, P, P, I, P, I, I, I, I, I, I, F, I, I, I, F, F, F, F, P]
     lib.ie_gemm_stream.restype = c_int
-    lib.ie_gemm_stream_tma.argtypes = [P, P, P, P, I, P, I, I, I, I, I, I, F, I, I, I, P, I, P, I, P, I, P]
+    lib.ie_gemm_stream_tma.argtypes = [P, P, P, P, I, P, I, I, I, I, I, I, F, I, I, I, P, I, P, I, P, I, F, F, F, F, P]
     lib.ie_gemm_stream_tma.restype = c_int
     lib.ie_gemm_stream_tma_supports.argtypes = [I, I, I, I]
     lib.ie_gemm_stream_tma_supports.restype = c_int
@@ -1292,13 +1341,14 @@ def gemm_stream_ring_supports(m: int, n: int, k: int, normed: bool) -> bool:
 
 def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, m: int, epi: str = "bf16",
                 gain: torch.Tensor | None = None, eps: float = 0.0, row_index: torch.Tensor | None = None,
-                nt: int | None = None, prenormed=None, normout=None, lib=None) -> None:
+                nt: int | None = None, prenormed=None, normout=None, lib=None, act: tuple | None = None) -> None:
     """c = a @ w^T for m <= 64 rows, bfloat16 weights, reading w once at HBM speed.
 
     With ``gain`` the input ``a`` is the float32 residual stream (rows gathered by ``row_index`` if given)
     and RMSNorm with that gain and ``eps`` is applied inside the kernel.  ``epi``: "bf16" or "f32" store,
     "residual" adds into the float32 ``c``, "silu_mul" takes w's rows as alternating gate/up and writes
-    silu(gate)*up, half as wide.
+    silu(gate)*up, half as wide; "glu" the same with the activation ``act`` of ``glu_constants``; "relu2" stores
+    max(product, 0)^2.
 
     Two products can hand a norm over between them.  ``normout=(xg, gain_next, ssq)`` with epi "residual":
     besides adding into ``c`` the kernel writes ``xg`` = bfloat16(new c * gain_next) and, per block, the sums of
@@ -1307,6 +1357,8 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, m: int, epi: 
     n, k = w.shape
     assert w.dtype is torch.bfloat16 and w.stride(1) == 1 and a.stride(-1) == 1 and c.stride(-1) == 1
     lib = lib or stream_library()
+    assert epi not in ("glu", "relu2") or (gain is None and prenormed is None)
+    act = _act4(act)
     if prenormed is not None or normout is not None:
         pro = 2 if prenormed is not None else 0
         xg, ssq = (prenormed if prenormed is not None else (normout[0], normout[2]))
@@ -1318,7 +1370,7 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, m: int, epi: 
         _check(lib.ie_gemm_stream_tma(_ptr(src), _ptr(w), _ptr(c), None, 0, None, m, n, k, src.stride(0), w.stride(0),
                                       c.stride(0), float(eps), pro, code, sm_count(), _ptr(xg), xg.stride(0),
                                       _ptr(gain_next), dtype_code(gain_next.dtype) if gain_next is not None else 0,
-                                      _ptr(ssq), ssq.shape[1], _stream()),
+                                      _ptr(ssq), ssq.shape[1], *act, _stream()),
                f"gemm_stream_tma(m={m}, n={n}, k={k}, {epi}, handed-over norm)")
         return
     if gain is None:
@@ -1331,7 +1383,7 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, m: int, epi: 
                                       dtype_code(gain.dtype) if gain is not None else 0, _ptr(row_index), m, n, k,
                                       a.stride(0), w.stride(0), c.stride(0), float(eps),
                                       0 if gain is None else 1, _EPI[epi], sm_count(), None, 0, None, 0, None, 0,
-                                      _stream()),
+                                      *act, _stream()),
                f"gemm_stream_tma(m={m}, n={n}, k={k}, {epi})")
         return
     if nt is None:
@@ -1341,7 +1393,7 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, m: int, epi: 
     _check(lib.ie_gemm_stream(_ptr(a), _ptr(w), _ptr(c), _ptr(gain),
                                            dtype_code(gain.dtype) if gain is not None else 0, _ptr(row_index), m, n, k,
                                            a.stride(0), w.stride(0), c.stride(0), float(eps),
-                                           0 if gain is None else 1, _EPI[epi], nt, _stream()),
+                                           0 if gain is None else 1, _EPI[epi], nt, *act, _stream()),
            f"gemm_stream(m={m}, n={n}, k={k}, {epi})")
 
 
@@ -1356,7 +1408,7 @@ def tcgen05_library():
         P, I = c_void_p, c_int
         lib.ie_gemm_tcgen05.argtypes = [P, P, P, I, I, I, I, I, I, I, I, I, P]
         lib.ie_gemm_tcgen05.restype = c_int
-        lib.ie_gemm_tcgen05_act.argtypes = [c_void_p] * 3 + [c_int] * 10 + [c_float] * 3 + [c_void_p]
+        lib.ie_gemm_tcgen05_act.argtypes = [c_void_p] * 3 + [c_int] * 10 + [c_float] * 4 + [c_void_p]
         lib.ie_gemm_tcgen05_act.restype = c_int
         lib.ie_gemm_tcgen05_supports.argtypes = [I, I, I, I, I]
         lib.ie_gemm_tcgen05_supports.restype = c_int
@@ -1375,20 +1427,20 @@ def gemm_tcgen05_error() -> int:
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epi: str = "bf16", bn: int = 256,
-                 act: tuple[float, float, float] | None = None) -> None:
+                 act: tuple | None = None) -> None:
     """c = a @ w^T on the fifth-generation tensor cores (TMA operands, accumulator in tensor memory).
 
     ``epi``: "bf16" store, "residual" adds into the float32 ``c``, "silu_mul" takes w's rows as alternating
-    gate/up and writes silu(gate)*up, half as wide.  ``bn``: tile width, 128 or 256.  ``act`` = (alpha, limit, up_offset)
-    with "silu_mul": g' sigmoid(alpha g') (u' + up_offset) with g' = min(g, limit) and u' = clamp(u, -limit, limit)."""
+    gate/up and writes silu(gate)*up, half as wide, "relu2" stores max(product, 0)^2.  ``bn``: tile width, 128 or 256.
+    ``act`` with "silu_mul": the activation of ``glu_constants`` instead of silu."""
     m, k = a.shape
     n = w.shape[0]
     assert a.dtype is torch.bfloat16 and w.dtype is torch.bfloat16 and a.stride(1) == 1 and w.stride(1) == 1
     assert act is None or epi == "silu_mul"
-    alpha, limit, up_offset = act if act is not None else (1.0, 0.0, 0.0)
+    alpha, limit, up_offset, cubic = _act4(act)
     _check(tcgen05_library().ie_gemm_tcgen05_act(_ptr(a), _ptr(w), _ptr(c), m, n, k, a.stride(0), w.stride(0), c.stride(0),
                                                  _EPI[epi], bn, sm_count(), 1 if act is not None else 0, float(alpha),
-                                                 float(limit), float(up_offset), _stream()),
+                                                 float(limit), float(up_offset), float(cubic), _stream()),
            f"gemm_tcgen05(m={m}, n={n}, k={k}, {epi})")
 
 

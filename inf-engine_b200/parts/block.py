@@ -1,7 +1,8 @@
 """Residual blocks.  The pre-norm block: ``x += mixer(norm(x)); x += ff(norm(x))``
 (engine/llama_block.py:50-62); beside it a block that norms its sublayers' outputs, a pre-norm block with gates per
-coordinate, and a block with a norm before and after each sublayer whose mixer may read shifted inputs, and a pre-norm block whose
-sublayers' results take a multiplier per coordinate.  The sums are folded into the norm that follows
+coordinate, a block with a norm before and after each sublayer whose mixer may read shifted inputs, a pre-norm block whose
+sublayers' results take a multiplier per coordinate, and a block whose two sublayers read one norm's output side by side.
+The sums are folded into the norm that follows
 them: a block hands on the residual and a delta that is not added yet.  A block
 whose spec has no feed-forward is the first half alone."""
 
@@ -340,8 +341,52 @@ class ScaledPreNormBlock:
             return residual, pending
         h = self.ff_norm.add_norm(residual, pending)
         unsummed = getattr(self.feedforward, "forward_unsummed", None)
-        y, weights = unsummed(h, ctx) if unsummed is not None else (self.feedforward.forward(h, ctx), None)
-        return residual, ScaledDelta(y, self.ff_scale, weights)
+        y, weights, more = unsummed(h, ctx) if unsummed is not None else (self.feedforward.forward(h, ctx), None, ())
+        return residual, ScaledDelta(y, self.ff_scale, weights, extras=more)
+
+
+@register_block("parallel")
+class ParallelBlock:
+    """``x += c * (mixer(h) + ff(h))`` with h = norm(x): one norm, whose output both sublayers read.  Neither result is
+    summed up here: the mixer's, the feed-forward's (for a mixture of experts the chosen experts' rows, their weights and a
+    shared expert's row), the constant, the sum into the float32 residual and the norm that comes next are one kernel (a
+    norm that takes a ``ScaledDelta``).  A block without a feed-forward is ``x += c * mixer(h)``."""
+
+    @staticmethod
+    def expected_tensors(spec):
+        out = {}
+        out.update(norm_class(spec.mixer_norm).expected_tensors(spec.mixer_norm))
+        out.update(mixer_class(spec.mixer).expected_tensors(spec.mixer))
+        if spec.feedforward is not None:
+            out.update(feedforward_class(spec.feedforward).expected_tensors(spec.feedforward))
+        return out
+
+    def __init__(self, spec, tensors, rt):
+        if spec.ff_norm is not None:
+            raise ValueError("a block whose sublayers read one norm's output has no norm of the feed-forward's own")
+        self.spec = spec
+        self.mixer_norm = build_norm(spec.mixer_norm, tensors, rt)
+        self.mixer = build_mixer(spec.mixer, tensors, rt)
+        self.feedforward = build_feedforward(spec.feedforward, tensors, rt) if spec.feedforward is not None else None
+        self.mult = float(spec.residual_mult)
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(p, "graph_safe", False) for p in (self.mixer, self.feedforward) if p is not None)
+
+    def forward(self, residual, pending, ctx, cache):
+        ctx.handover = None
+        ctx.upcoming_norm = None
+        ctx.residual_cast = None
+        h = self.mixer_norm.add_norm(residual, pending)
+        a = self.mixer.forward(h, ctx, cache)
+        if self.feedforward is None:
+            return residual, ScaledDelta(a, mult=self.mult)
+        unsummed = getattr(self.feedforward, "forward_unsummed", None)
+        if unsummed is None:
+            return residual, ScaledDelta(a, mult=self.mult, extras=(self.feedforward.forward(h, ctx),))
+        y, weights, more = unsummed(h, ctx)
+        return residual, ScaledDelta(y, None, weights, self.mult, (a,) + tuple(more))
 
 
 def _fuses(part, n_tokens: int, norm) -> bool:

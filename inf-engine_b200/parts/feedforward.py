@@ -2,8 +2,11 @@
 gate, clamps of both branches and an offset of the up branch are options of the spec (``kernels.glu_act``).
 
 Gate and up are one matrix product over the row-concatenated weights
-[2*intermediate, hidden]; the activation and the product by ``up`` are one
-kernel in float32 arithmetic.
+[2*intermediate, hidden]; the activation and the product by ``up`` ride in that
+product's epilogue (float32 arithmetic) in the kernels for few rows and for many,
+and are one kernel beside the library product.
+
+``MLP``: ``down(act(up(x)))`` without a gate, the activation in the first product's epilogue in the same way.
 
 ``PolyNormMLP``: ``down(act(up(x) + b_up)) + b_down`` with the PolyNorm activation,
 a polynomial of the normalised first three powers of each token's hidden vector
@@ -18,6 +21,9 @@ from .. import kernels
 from ..weights.loader import ExpectedTensor
 from .linear import Linear, stream_into_residual, stream_normed
 from .registry import register_feedforward
+
+
+MLP_ACTIVATIONS = ("relu2",)      # activations of a feed-forward without a gate
 
 
 @register_feedforward("gated_mlp")
@@ -35,7 +41,7 @@ class GatedMLP:
     def __init__(self, spec, tensors, rt):
         if spec.activation not in kernels.GLU_KINDS:
             raise ValueError(f"activation {spec.activation!r} is not built (known: {sorted(kernels.GLU_KINDS)})")
-        # the products' fused epilogues know silu(gate) * up only; any other activation is a kernel of its own
+        # the product with a norm in its prologue knows silu(gate) * up only
         self.plain_silu = spec.activation == "silu" and spec.up_offset == 0.0
         self.spec = spec
         self.rt = rt
@@ -45,6 +51,7 @@ class GatedMLP:
         both = torch.stack([gate.to(dtype), up.to(dtype)], dim=1).reshape(2 * spec.intermediate, spec.hidden)
         self.gate_up = Linear(both.contiguous(), rt, "gate_up")
         self.down = Linear(tensors[spec.down_proj], rt, "down")
+        self.act = kernels.glu_constants(spec.activation, spec.act_alpha, spec.act_limit, spec.up_offset)
 
     def can_fuse(self, n_tokens: int, norm) -> bool:
         return (self.plain_silu and hasattr(norm, "fusable_rms") and self.gate_up.streams(n_tokens, normed=True)
@@ -70,9 +77,10 @@ class GatedMLP:
                 and kernels.gemm_tcgen05_supports(n, 2 * s.intermediate, s.hidden, x.stride(0), w.stride(0))):
             # gate/up on the tcgen05 tensor cores with the gated activation in the epilogue: the [n, 2*intermediate]
             # matrix never goes to memory
-            act = None if self.plain_silu else \
-                ((s.act_alpha, s.act_limit, s.up_offset) if s.activation == "clamped_swish" else (1.0, float("inf"), s.up_offset))
-            kernels.gemm_tcgen05(x, w, h, "silu_mul", act=act)
+            kernels.gemm_tcgen05(x, w, h, "silu_mul", act=None if self.plain_silu else self.act)
+        elif not self.plain_silu and self.gate_up.streams(n) and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+            # a few rows (decode tokens): the weight-streaming product with the activation in its epilogue
+            self.gate_up.stream(x, h, n, "glu", act=self.act)
         else:
             gu = self.gate_up(x, ws.take("ff_gate_up", (n, 2 * s.intermediate), dt))
             if self.plain_silu:
@@ -81,6 +89,39 @@ class GatedMLP:
                 kernels.glu_act(gu, h, s.activation, interleaved=True, alpha=s.act_alpha, limit=s.act_limit,
                                 up_offset=s.up_offset)
         return self.down(h, ws.take("ff_out", (n, s.hidden), dt))
+
+
+@register_feedforward("mlp")
+class MLP:
+    graph_safe = True
+
+    @staticmethod
+    def expected_tensors(spec):
+        return {spec.up_proj: ExpectedTensor((spec.intermediate, spec.hidden)),
+                spec.down_proj: ExpectedTensor((spec.hidden, spec.intermediate))}
+
+    def __init__(self, spec, tensors, rt):
+        if spec.activation not in MLP_ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not built (known: {', '.join(MLP_ACTIVATIONS)})")
+        self.spec = spec
+        self.rt = rt
+        self.up = Linear(tensors[spec.up_proj].contiguous(), rt, "up")
+        self.down = Linear(tensors[spec.down_proj].contiguous(), rt, "down")
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        n = x.shape[0]
+        s, ws, dt = self.spec, self.rt.ws, self.rt.act_dtype
+        h = ws.take("mlp_hidden", (n, s.intermediate), dt)
+        w = self.up.weight
+        if (dt is torch.bfloat16 and w.dtype is torch.bfloat16 and n >= GatedMLP.TCGEN05_MIN_ROWS
+                and kernels.gemm_tcgen05_supports(n, s.intermediate, s.hidden, x.stride(0), w.stride(0))):
+            kernels.gemm_tcgen05(x, w, h, "relu2")
+        elif self.up.streams(n) and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+            self.up.stream(x, h, n, "relu2")
+        else:
+            self.up(x, h)
+            kernels.relu2(h, h)
+        return self.down(h, ws.take("mlp_out", (n, s.hidden), dt))
 
 
 @register_feedforward("polynorm_mlp")

@@ -6,6 +6,8 @@ RMS-normed) and a rotated key part that all heads share.  A head's unrotated key
 carried over to the compressed space once (a product per head, ``heads_product``), every head then reads the SAME
 cached rows (attention with one key head whose values are the first ``kv_rank`` dimensions of its keys), and the
 head's output ``v_up_h (sum_j w_j c_j)`` is one more product per head.  Nothing per head is ever stored per token.
+A layer without a ``down_proj`` compresses nothing: it reads the rows that another run's cache holds (it writes none and
+asks for no pages), with its own queries and its own way into and out of the compressed space.
 
 ``DifferentialAttention``: the two maps of a head are attention heads of their own that share a value head: 2 x heads
 query heads over 2 x kv_heads key heads and kv_heads value heads.  The query rows are reordered once at load
@@ -137,8 +139,11 @@ class LatentAttention:
             out[spec.q_norm] = ExpectedTensor((spec.q_rank,), init="gain")
         out.update({
             spec.q_proj: ExpectedTensor((spec.n_heads * qd, spec.q_rank or spec.hidden)),
-            spec.down_proj: ExpectedTensor((spec.kv_rank + spec.rot_dim, spec.hidden)),
-            spec.latent_norm: ExpectedTensor((spec.kv_rank,), init="gain"),
+        })
+        if spec.down_proj:
+            out[spec.down_proj] = ExpectedTensor((spec.kv_rank + spec.rot_dim, spec.hidden))
+            out[spec.latent_norm] = ExpectedTensor((spec.kv_rank,), init="gain")
+        out.update({
             spec.k_up: ExpectedTensor((spec.n_heads * spec.head_dim, spec.kv_rank)),
             spec.v_up: ExpectedTensor((spec.n_heads * spec.v_head_dim, spec.kv_rank)),
         })
@@ -168,7 +173,12 @@ class LatentAttention:
         self.q_rank = int(spec.q_rank or 0)
         if self.q_rank and r:
             raise NotImplementedError("queries through a compressed vector together with a rotated part are not built")
-        ws = [tensors[spec.q_down] if self.q_rank else tensors[spec.q_proj], tensors[spec.down_proj]]
+        self.borrows = not spec.down_proj          # reads another run's rows
+        if self.borrows and (self.q_rank or r):
+            raise NotImplementedError("a layer that reads another's compressed vectors has plain queries without a rotated part")
+        ws = [tensors[spec.q_down] if self.q_rank else tensors[spec.q_proj]]
+        if not self.borrows:
+            ws.append(tensors[spec.down_proj])
         if spec.head_gate is not None:
             ws.append(tensors[spec.head_gate])
         stacked, self.cols = stack_rows(ws, _common_dtype(ws))
@@ -176,7 +186,8 @@ class LatentAttention:
         self.q_width = H * self.q_dim
         self.first_width = self.q_rank or self.q_width
         self.gate_width = H if spec.head_gate is not None else 0
-        self.latent_gain = tensors[spec.latent_norm].contiguous()
+        self.gate_col = self.cols[-2] if self.gate_width else 0
+        self.latent_gain = tensors[spec.latent_norm].contiguous() if not self.borrows else None
         if self.q_rank:
             self.q_up = Linear(tensors[spec.q_proj], rt, "latent_q_up")
             self.q_gain = tensors[spec.q_norm].contiguous()
@@ -196,6 +207,8 @@ class LatentAttention:
 
     def cache_requirement(self) -> CacheRequirement:
         s = self.spec
+        if self.borrows:
+            raise ValueError("a layer that compresses nothing itself must read the cache of an earlier run (cache_from)")
         return CacheRequirement(kind="kv", n_kv_heads=1, head_dim=self.row_dim, v_head_dim=s.kv_rank, dtype=self.rt.act_dtype,
                                 values_in_keys=True, chunk=s.chunk, window=s.window)
 
@@ -205,11 +218,14 @@ class LatentAttention:
         H, kr = s.n_heads, s.kv_rank
         cols = self.cols
         proj = self.proj(x, rt.ws.take("latent_proj", (n, cols[-1]), rt.act_dtype))
-        q, row = proj[:, :self.first_width], proj[:, cols[1]:cols[1] + self.row_dim]
+        q = proj[:, :self.first_width]
+        row = proj[:, cols[1]:cols[1] + self.row_dim] if not self.borrows else None
         kvctx = ctx.kv[cache.group]
         inv_freq, rot_dims, neighbours, mult = _rotation(self.position)
         kpool = cache.k if cache.write else None
-        if self.q_rank:
+        if self.borrows:
+            pass                                   # the rows lie in the cache already, those of this step's tokens too
+        elif self.q_rank:
             # the norms of both compressed vectors and the cache write (the queries' vector is one "head" of q_rank
             # numbers here), then the queries' expansion
             kernels.head_prepare(q, 1, self.q_rank, row, 1, self.row_dim, ctx.positions, kvctx.slot_mapping, kpool,
@@ -218,7 +234,8 @@ class LatentAttention:
             q = self.q_up(q, rt.ws.take("latent_q", (n, self.q_width), rt.act_dtype))
         else:
             # norm of the compressed part, rotation of the shared key part and of every head's rotated part, cache write
-            kernels.head_prepare(q, H, self.q_dim, row, 1, self.row_dim, ctx.positions, kvctx.slot_mapping, kpool,
+            # (queries without a rotated part pass as they are: no query heads for the kernel)
+            kernels.head_prepare(q, H if rot_dims else 0, self.q_dim, row, 1, self.row_dim, ctx.positions, kvctx.slot_mapping, kpool,
                                  ctx.page_size, k_gain=self.latent_gain, k_norm_dims=kr, eps=s.norm_eps,
                                  inv_freq=inv_freq, rot_dims=rot_dims, q_rot_off=s.head_dim, k_rot_off=kr,
                                  neighbours=neighbours, mult=mult)
@@ -231,7 +248,7 @@ class LatentAttention:
         heads_product(mixed, kr, self.expand, heads, s.v_head_dim)
         if self.gate_width:
             # a head's output times sigmoid of its gate
-            kernels.gate_mul(heads, proj[:, cols[2]:cols[2] + H], group=s.v_head_dim)
+            kernels.gate_mul(heads, proj[:, self.gate_col:self.gate_col + H], group=s.v_head_dim)
         return self.o(heads, rt.ws.take("mixer_out", (n, s.hidden), rt.act_dtype))
 
 

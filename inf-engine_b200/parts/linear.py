@@ -63,9 +63,9 @@ class Linear:
         return True
 
     def stream(self, x: torch.Tensor, out: torch.Tensor, n_rows: int, epi: str = "bf16", gain=None, eps: float = 0.0,
-               row_index=None) -> torch.Tensor:
+               row_index=None, act=None) -> torch.Tensor:
         """The product through the weight-streaming kernel, with its fused prologue and epilogue."""
-        kernels.gemm_stream(x, self.weight, out, n_rows, epi, gain, eps, row_index)
+        kernels.gemm_stream(x, self.weight, out, n_rows, epi, gain, eps, row_index, act=act)
         return out
 
     def __call__(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:

@@ -93,7 +93,10 @@ class DecoderModel:
         return residual, pending
 
     def finish_logits(self, logits: torch.Tensor, ctx) -> torch.Tensor:
-        """What a derived top level does to the head's float32 logits (in place) before they leave; nothing here."""
+        """What is done to the head's float32 logits (in place) before they leave: the cap, if the spec has one; a derived
+        top level may do more."""
+        if self.spec.logit_softcap is not None:
+            kernels.softcap(logits, self.spec.logit_softcap)
         return logits
 
     def forward(self, ctx) -> torch.Tensor | None:

@@ -7,6 +7,8 @@ that precedes it in a pre-norm block (engine/llama_block.py:53-62).  With
 sublayers' OUTPUTS: the normed rows are added into the residual.
 ``GroupedRMSNorm`` norms each of several equal consecutive parts of the row by itself, and takes a summand that carries
 a multiplier per coordinate or is a mixture of experts not summed up yet (``ScaledDelta``) in the same kernel.
+``TanhNorm`` (dynamic tanh) has no statistics: ``tanh(alpha x) * gain + bias``, coordinate by coordinate, with such a summand
+taken in the same way.
 LayerNorm: ``(x - mean) / sqrt(variance + eps) * weight + bias`` with the variance
 the mean of the squared deviations, the same way."""
 
@@ -20,19 +22,22 @@ from .registry import register_norm
 
 
 class ScaledDelta:
-    """A summand of the residual stream that is not added yet: ``scale * y`` with ``scale`` float32 [d] (None: 1), or
-    ``scale * sum_r weights[n, r] * y[n * top + r]`` with ``weights`` float32 [n, top]."""
+    """A summand of the residual stream that is not added yet: ``mult * scale * (y + sum of extras)`` with ``scale``
+    float32 [d] (None: 1), or, with ``weights`` float32 [n, top], ``sum_r weights[n, r] * y[n * top + r]`` in the place of
+    y.  ``extras``: up to two results of sublayers that read the same input, of one type."""
 
-    __slots__ = ("y", "scale", "weights")
+    __slots__ = ("y", "scale", "weights", "mult", "extras")
 
-    def __init__(self, y: torch.Tensor, scale: torch.Tensor | None = None, weights: torch.Tensor | None = None):
-        self.y, self.scale, self.weights = y, scale, weights
+    def __init__(self, y: torch.Tensor, scale: torch.Tensor | None = None, weights: torch.Tensor | None = None,
+                 mult: float = 1.0, extras: tuple = ()):
+        self.y, self.scale, self.weights, self.mult, self.extras = y, scale, weights, mult, extras
 
 
 def add_pending(residual: torch.Tensor, pending) -> None:
     """residual += pending, a tensor or a ``ScaledDelta``."""
     if isinstance(pending, ScaledDelta):
-        kernels.stream_norm(residual, pending.y, pending.scale, pending.weights, None, 1, 0.0, None)
+        kernels.stream_norm(residual, pending.y, pending.scale, pending.weights, None, 1, 0.0, None, mult=pending.mult,
+                            extras=pending.extras)
     else:
         kernels.residual_add(residual, pending)
 
@@ -116,7 +121,40 @@ class GroupedRMSNorm:
 
     def _norm(self, residual, delta, out, row_index=None):
         d = delta if isinstance(delta, ScaledDelta) else ScaledDelta(delta)
-        kernels.stream_norm(residual, d.y, d.scale, d.weights, self.gain, self.groups, self.eps, out, row_index)
+        kernels.stream_norm(residual, d.y, d.scale, d.weights, self.gain, self.groups, self.eps, out, row_index,
+                            mult=d.mult, extras=d.extras)
+        return out
+
+    def add_norm(self, residual: torch.Tensor, delta, out_name: str = "normed") -> torch.Tensor:
+        return self._norm(residual, delta, self.rt.ws.take(out_name, tuple(residual.shape), self.rt.act_dtype))
+
+    def gather_norm(self, residual: torch.Tensor, delta, row_index: torch.Tensor, n_rows: int,
+                    out_name: str = "normed_rows") -> torch.Tensor:
+        return self._norm(residual, delta, self.rt.ws.take(out_name, (n_rows, self.size), self.rt.act_dtype), row_index)
+
+
+@register_norm("tanh_norm")
+class TanhNorm:
+    """Dynamic tanh: ``tanh(alpha x) * gain + bias``, coordinate by coordinate, alpha one number of the model's."""
+
+    @staticmethod
+    def expected_tensors(spec):
+        return {spec.weight: ExpectedTensor((spec.size,), init="gain"), spec.bias: ExpectedTensor((spec.size,)),
+                spec.alpha: ExpectedTensor((), init="gain")}
+
+    def __init__(self, spec, tensors, rt):
+        self.spec = spec
+        self.rt = rt
+        self.gain, self.bias = tensors[spec.weight].contiguous(), tensors[spec.bias].contiguous()
+        if self.gain.dtype != self.bias.dtype:
+            self.gain, self.bias = self.gain.float(), self.bias.float()
+        self.tanh = (float(tensors[spec.alpha].float()), self.bias)
+        self.size = spec.size
+
+    def _norm(self, residual, delta, out, row_index=None):
+        d = delta if isinstance(delta, ScaledDelta) else ScaledDelta(delta)
+        kernels.stream_norm(residual, d.y, d.scale, d.weights, self.gain, 1, 0.0, out, row_index, mult=d.mult,
+                            extras=d.extras, tanh=self.tanh)
         return out
 
     def add_norm(self, residual: torch.Tensor, delta, out_name: str = "normed") -> torch.Tensor:

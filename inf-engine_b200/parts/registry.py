@@ -21,8 +21,9 @@ Mixer           expected_tensors(spec); __init__(spec, tensors, rt)
                 graph_safe: bool   (True when forward reads batch metadata on the device only)
 FeedForward     expected_tensors(spec); __init__(spec, tensors, rt); forward(x, ctx) -> [N, hidden]
                 graph_safe: bool   (as for a mixer; a part that does not say so keeps decode steps out of graphs)
-                forward_unsummed (optional): forward_unsummed(x, ctx) -> (y, weights) in place of forward, for a block
-                    that forms ``sum_r weights[n, r] * y[n * top + r]`` as it adds the result to the residual
+                forward_unsummed (optional): forward_unsummed(x, ctx) -> (y, weights, more) in place of forward, for a
+                    block that forms ``sum_r weights[n, r] * y[n * top + r]`` plus the rows of ``more`` (a tuple) as it
+                    adds the result to the residual
 Block           expected_tensors(spec); __init__(spec, tensors, rt)
                 graph_safe: bool   (every part of it is)
                 forward(residual, pending, ctx, cache) -> (residual, pending)
