@@ -490,6 +490,29 @@ def _nurilorn_configs(size):
 NURILORN_CAP = 30.0
 
 
+def _nurasun_configs(size):
+    """A Nurasun model of the size's width (attention in chunks of 1,024 positions whose values are its keys, a latent
+    layer, a latent layer that reads the former's vectors, attention again; dense feed-forwards of four times the width in
+    the first and third layer, 16 experts of which a token runs four beside a shared one in the others: as many ACTIVE
+    feed-forward parameters) and a Fovunex model of equal width, depth and head geometry with as many layers of each kind
+    (two-map attention in chunks, latent attention), the closest family the engine had."""
+    from inf_engine_b200.config import parse_config_dict
+    z = FAMILY_SIZES[size]
+    w, H, G, inter = z["width"], z["heads"], z["kv"], z["inter"]
+    dense = {"kind": "dense", "ff": inter}
+    moe = {"kind": "moe", "expert": {"ff": inter // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": inter // 2}}
+    att = {"heads": H, "kv_heads": G, "dim": FAMILY_HD, "vdim": FAMILY_HD, "scale": FAMILY_HD ** -0.5,
+           "rot": {"base": 10000.0, "dims": FAMILY_HD}, "mask": {"size": FOVUNEX_CHUNK}}
+    lat = {"heads": H, "dim": FAMILY_HD, "vdim": FAMILY_HD, "kv_rank": FOVUNEX_RANK, "scale": FAMILY_HD ** -0.5}
+    layers = [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "latent_attention", "mixer": lat, "mlp": moe},
+              {"type": "latent_attention", "mixer": dict(lat, kv_from=1), "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe}]
+    sun = parse_config_dict({"architecture": "Nurasun", "vocab": FAMILY_VOCAB, "width": w, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+                             "logit_softcap": 30.0, "layers": layers})
+    fvx = _fovunex_configs(size)[0].to_hf_dict()
+    _, diff, _, latent = fvx["layers"]
+    return sun, parse_config_dict(dict(fvx, layers=[diff, latent, latent, diff]))
+
+
 def _weight_bytes(runner):
     seen, n = set(), 0
     import torch
@@ -515,8 +538,8 @@ def run_family(args):
     from inf_engine_b200 import Engine, StepEntry, SamplingConfig, kernels
     from inf_engine_b200.sampling import pack_rows, request_key
 
-    if args.family not in ("barerax", "kipezen", "fovunex", "gavatar", "nurilorn"):
-        print(f"--family {args.family}: unknown (known: barerax, kipezen, fovunex, gavatar, nurilorn)")
+    if args.family not in ("barerax", "kipezen", "fovunex", "gavatar", "nurilorn", "nurasun"):
+        print(f"--family {args.family}: unknown (known: barerax, kipezen, fovunex, gavatar, nurilorn, nurasun)")
         return 2
     pk = peaks()
     torch.cuda.set_device(0)
@@ -1395,8 +1418,170 @@ def run_family(args):
             timed(lambda: kernels.gemm_tcgen05(x, dense_w, dense_out, "silu_mul")), flops=2 * N * 2 * inter * W)
         return rows
 
+    def nurasun_kernel_table(size):
+        """Every kernel that the Nurasun family added or extended, alone, beside the like kernel of the closest family that
+        has one (Fovunex; its feed-forward is dense, so the experts' kernels stand beside Kipezen's), at 2,048 tokens of one
+        request and at 8 requests of one token over 2,048 keys."""
+        from inf_engine_b200.engine.batch import KVGroupContext, StepContext
+        from inf_engine_b200.parts import Runtime
+        from inf_engine_b200.parts.latent import attend_float32, heads_product
+        z = FAMILY_SIZES[size]
+        W, H, G, hd, inter = z["width"], z["heads"], z["kv"], FAMILY_HD, z["inter"]
+        N, B, dev, bf = PROMPT_LEN, 8, "cuda", torch.bfloat16
+        g = torch.Generator(device=dev).manual_seed(1)
+        rnd = lambda *shape: (torch.randn(*shape, device=dev, generator=g) * 0.5)
+        i32 = lambda v: torch.as_tensor(v, dtype=torch.int32, device=dev)
+        rows = []
+
+        def add(name, like, ms, ms_like, nbytes=None, nbytes_like=None, flops=None, flops_like=None, note=None):
+            rec = {"kernel": name, "like": like, "ms": ms, "like_ms": ms_like}
+            if nbytes is not None:
+                rec["frac_of_hbm"] = nbytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"]
+                rec["like_frac_of_hbm"] = (nbytes_like or nbytes) / (ms_like * 1e-3) / 1e9 / pk["hbm_gbs"]
+            if flops is not None:
+                rec["frac_of_bf16"] = flops / (ms * 1e-3) / 1e12 / pk["bf16_tflops"]
+                rec["like_frac_of_bf16"] = (flops_like or flops) / (ms_like * 1e-3) / 1e12 / pk["bf16_tflops"]
+            if note:
+                rec["note"] = note
+            rows.append(rec)
+
+        rt = Runtime(dev, bf)
+        n_pages = B * N // PAGE
+
+        def context(q_lens, before):
+            ctx = StepContext(rt, PAGE)
+            R, n = len(q_lens), sum(q_lens)
+            ctx.n_tokens, ctx.n_requests, ctx.n_logits = n, R, 0
+            starts = [0]
+            for ql in q_lens:
+                starts.append(starts[-1] + ql)
+            per = n_pages // R
+            ctx.q_start, ctx.ctx_before = i32(starts), i32(before)
+            ctx.positions = i32([b + t for ql, b in zip(q_lens, before) for t in range(ql)])
+            ctx.slots = i32(list(range(R)))
+            table_ = torch.arange(per * R, dtype=torch.int32, device=dev).view(R, per)
+            sm = i32([(r * per + (b + t) // PAGE) * PAGE + (b + t) % PAGE for r, (ql, b) in enumerate(zip(q_lens, before)) for t in range(ql)])
+            ctx.kv = [KVGroupContext(sm, table_)]
+            ctx.host = {"q_lens": list(q_lens), "ctx_before": list(before), "q_start": starts}
+            ctx.max_q_len, ctx.max_seq_len = max(q_lens), max(b + ql for ql, b in zip(q_lens, before))
+            ctx.keys_cap = ctx.max_seq_len
+            return ctx
+
+        ctx_p, ctx_d = context([N], [0]), context([1] * B, [N - 1] * B)
+        both = ((N, ctx_p, "prompt"), (B, ctx_d, "decode b8"))
+        pairs_all = N * (N + 1) // 2
+        pairs_c = (N // FOVUNEX_CHUNK) * FOVUNEX_CHUNK * (FOVUNEX_CHUNK + 1) // 2
+        # the stream: two sublayers' results, or the experts' rows, the mixer's and the shared expert's, and the norm
+        E, top, ffe, ffs = 16, 4, inter // 4, inter // 2
+        res, a, b, out = rnd(N, W), rnd(N, W).to(bf), rnd(N, W).to(bf), torch.empty(N, W, device=dev, dtype=bf)
+        pairs_y, wts = rnd(N * top, W), torch.rand(N, top, device=dev, generator=g)
+        gain, off = (1 + 0.1 * rnd(W)).to(bf), rnd(W).to(bf)
+        for n, _, what in both:
+            like = timed(lambda: (kernels.gated_residual_add(res[:n], a[:n], b[:n], off), kernels.rmsnorm(res[:n], None, gain, out[:n], 1e-5)))
+            nb_like = n * W * (4 + 4 + 2 + 2 + 4 + 2)
+            add(f"two sublayers' sum into the stream + dynamic tanh, {what}", "gated sum into the stream, norm (two kernels, one sublayer)",
+                timed(lambda: kernels.stream_norm(res[:n], a[:n], None, None, gain, 1, 0.0, out[:n], mult=0.5, extras=(b[:n],), tanh=(0.7, off))),
+                like, n * W * (4 + 4 + 2 + 2 + 2), nb_like)
+            add(f"experts' weighted sum + mixer + shared expert into the stream + dynamic tanh, {what}",
+                "gated sum into the stream, norm (two kernels, one sublayer)",
+                timed(lambda: kernels.stream_norm(res[:n], pairs_y[:n * top], None, wts[:n], gain, 1, 0.0, out[:n], mult=0.5,
+                                                  extras=(a[:n], b[:n]), tanh=(0.7, off))),
+                like, n * W * (4 + 4 + 4 * top + 2 + 2 + 2), nb_like)
+        # attention whose values are its keys: H heads of 64 over G, chunks | two maps of 64 over values of 128
+        Hd, Gd, dv = H // 2, G // 2, 2 * hd
+        qk, qb, kb = rnd(N, (H + G) * hd).to(bf), rnd(H * hd).to(bf), rnd(G * hd).to(bf)
+        q, kx = qk[:, :H * hd], qk[:, H * hd:]
+        kpool, vpool = torch.randn(n_pages, G, PAGE, hd, device=dev, generator=g).to(bf), torch.randn(n_pages, G, PAGE, hd, device=dev, generator=g).to(bf)
+        vpool2 = torch.randn(n_pages, Gd, PAGE, dv, device=dev, generator=g).to(bf)
+        qkv, hg = rnd(N, (H + G) * hd + Gd * dv).to(bf), (1 + 0.1 * rnd(hd)).to(bf)
+        inv = (10000.0 ** (-2.0 * torch.arange(hd // 2, dtype=torch.float64) / hd)).to(dev)
+        inv_half = (10000.0 ** (-2.0 * torch.arange(hd // 4, dtype=torch.float64) / (hd // 2))).to(dev)
+        heads_out, maps = torch.empty(N, H * hd, device=dev, dtype=bf), torch.empty(N, H * dv, device=dev, dtype=bf)
+        for n, ctx, what in both:
+            add(f"biases + rotation + keys and values (the keys) to the cache, {what}", "map norms + rotation in halves + cache write (two maps a head)",
+                timed(lambda: kernels.head_prepare(q[:n], H, hd, kx[:n], G, hd, ctx.positions, ctx.kv[0].slot_mapping, kpool, PAGE, inv_freq=inv,
+                                                   rot_dims=hd, q_bias=qb, k_bias=kb, tied=True, vpool=vpool)),
+                timed(lambda: kernels.head_prepare(qkv[:n, :H * hd], H, hd, qkv[:n, H * hd:(H + G) * hd], G, hd, ctx.positions, ctx.kv[0].slot_mapping,
+                                                   kpool, PAGE, q_gain=hg, q_norm_dims=hd, k_gain=hg, k_norm_dims=hd, eps=1e-5, inv_freq=inv_half,
+                                                   rot_dims=hd // 2, v=qkv[:n, (H + G) * hd:], vpool=vpool2, n_v_heads=Gd, v_head_dim=dv)),
+                n * (H * 2 + G * 3) * hd * 2, n * ((H + G) * hd * 2 + 2 * Gd * dv) * 2)
+        # (positions 1,023 of a chunk: every key of it is visible)
+        att = lambda ctx, n: attend_float32(q[:n], heads_out[:n], kpool, vpool, ctx, ctx.kv[0], H, G, hd, hd, hd ** -0.5, FOVUNEX_CHUNK)
+        att2 = lambda ctx, n: attend_float32(q[:n], maps[:n], kpool, vpool2, ctx, ctx.kv[0], H, G, hd, dv, hd ** -0.5, FOVUNEX_CHUNK, n_v_heads=Gd)
+        add("attention in chunks of 1,024, prompt (%d heads over %d)" % (H, G), "attention in chunks, prompt (two maps a head, values of 128)",
+            timed(lambda: att(ctx_p, N), reps=5), timed(lambda: att2(ctx_p, N), reps=5), flops=4 * H * hd * pairs_c, flops_like=2 * H * (hd + dv) * pairs_c)
+        add("attention in chunks of 1,024, decode b8 (1,024 visible)", "attention in chunks, decode (two maps a head, 1,024 visible)",
+            timed(lambda: att(ctx_d, B)), timed(lambda: att2(ctx_d, B)), B * FOVUNEX_CHUNK * G * hd * 2 * 2, B * FOVUNEX_CHUNK * (G * hd + Gd * dv) * 2)
+        # latent attention: rows of 192 | rows of 192 and 64 rotated
+        kr, r = FOVUNEX_RANK, FOVUNEX_ROT
+        ql, row, lpool = rnd(N, H * (hd + r)).to(bf), rnd(N, kr + r).to(bf), torch.randn(n_pages, 1, PAGE, kr, device=dev, generator=g).to(bf)
+        lpool2 = torch.randn(n_pages, 1, PAGE, kr + r, device=dev, generator=g).to(bf)
+        lg = (1 + 0.1 * rnd(kr)).to(bf)
+        inv_l = (10000.0 ** (-2.0 * torch.arange(r // 2, dtype=torch.float64) / r)).to(dev)
+        absorb, absorb2, expand = (rnd(H, hd, kr) * 0.1).to(bf), (rnd(H, hd + r, kr + r) * 0.1).to(bf), (rnd(H, kr, hd) * 0.1).to(bf)
+        qc, qc2, mixed = (torch.empty(N, H * k_, device=dev, dtype=bf) for k_ in (kr, kr + r, kr))
+        qp, rp = rnd(N, H * hd).to(bf), rnd(N, kr).to(bf)
+        lat = lambda ctx, n: attend_float32(qc[:n], mixed[:n], lpool, lpool, ctx, ctx.kv[0], H, 1, kr, kr, 0.125, None, n_v_heads=1, v_row=kr)
+        lat2 = lambda ctx, n: attend_float32(qc2[:n], mixed[:n], lpool2, lpool2, ctx, ctx.kv[0], H, 1, kr + r, kr, 0.125, None, n_v_heads=1, v_row=kr + r)
+        for n, ctx, what in both:
+            add(f"compressed-row norm + cache write, {what}", "compressed-row norm + rotation of neighbours + cache write",
+                timed(lambda: kernels.head_prepare(qp[:n], 0, hd, rp[:n], 1, kr, ctx.positions, ctx.kv[0].slot_mapping, lpool, PAGE, k_gain=lg,
+                                                   k_norm_dims=kr, eps=1e-5)),
+                timed(lambda: kernels.head_prepare(ql[:n], H, hd + r, row[:n], 1, kr + r, ctx.positions, ctx.kv[0].slot_mapping, lpool2, PAGE,
+                                                   k_gain=lg, k_norm_dims=kr, eps=1e-5, inv_freq=inv_l, rot_dims=r, q_rot_off=hd, k_rot_off=kr,
+                                                   neighbours=True, mult=1.1)),
+                n * kr * 2 * 2, n * (H * (hd + r) * 2 + (kr + r) * 2) * 2)
+            kw = (lambda f, f2: dict(flops=n * f, flops_like=n * f2)) if n == N else (lambda f, f2: dict(nbytes=f, nbytes_like=f2))   # (bytes of the weights)
+            add(f"queries into the compressed space, a product a head, {what}", "the same with a rotated part",
+                timed(lambda: heads_product(qp[:n], hd, absorb, qc[:n], kr)), timed(lambda: heads_product(ql[:n], hd + r, absorb2, qc2[:n], kr + r)),
+                **kw(2 * H * hd * kr, 2 * H * (hd + r) * (kr + r)))
+            add(f"values out of the compressed space, a product a head, {what}", "the same", *[timed(lambda: heads_product(mixed[:n], kr, expand, heads_out[:n], hd))] * 2,
+                **kw(2 * H * hd * kr, 2 * H * hd * kr))
+            kw = dict(flops=4 * H * kr * pairs_all, flops_like=2 * H * (2 * kr + r) * pairs_all) if n == N else dict(nbytes=B * N * kr * 2, nbytes_like=B * N * (kr + r) * 2)
+            add(f"latent attention, {what} ({H} heads over one row of {kr}, every key)", f"latent attention (rows of {kr + r})",
+                timed(lambda: lat(ctx, n), reps=5), timed(lambda: lat2(ctx, n), reps=5), **kw)
+        # feed-forwards
+        x = rnd(N, W).to(bf)
+        gelu, clamped = kernels.glu_constants("gelu_tanh"), kernels.glu_constants("clamped_swish", 1.702, 7.0, 1.0)
+        dense_w, hidden = (rnd(2 * inter, W) * 0.1).to(bf), torch.empty(N, inter, device=dev, dtype=bf)
+        add("dense gate/up product with the tanh form of gelu, prompt", "dense gate/up product with the clamped activation",
+            timed(lambda: kernels.gemm_tcgen05(x, dense_w, hidden, "silu_mul", act=gelu)),
+            timed(lambda: kernels.gemm_tcgen05(x, dense_w, hidden, "silu_mul", act=clamped)), flops=2 * N * 2 * inter * W)
+        add("dense gate/up product with the tanh form of gelu, decode b8", "dense gate/up product with silu (the Llama path)",
+            timed(lambda: kernels.gemm_stream(x[:B], dense_w, hidden[:B], B, "glu", act=gelu)),
+            timed(lambda: kernels.gemm_stream(x[:B], dense_w, hidden[:B], B, "silu_mul")), 2 * inter * W * 2)
+        shared_w, sh = (rnd(ffs, W) * 0.1).to(bf), torch.empty(N, ffs, device=dev, dtype=bf)
+        add("shared expert's first product with the square of relu, prompt", "the product alone",
+            timed(lambda: kernels.gemm_tcgen05(x, shared_w, sh, "relu2")), timed(lambda: kernels.gemm_tcgen05(x, shared_w, sh, "bf16")), flops=2 * N * ffs * W)
+        add("shared expert's first product with the square of relu, decode b8", "the product alone",
+            timed(lambda: kernels.gemm_stream(x[:B], shared_w, sh[:B], B, "relu2")), timed(lambda: kernels.gemm_stream(x[:B], shared_w, sh[:B], B)), ffs * W * 2)
+        logits = rnd(N, E + 1) * 2
+        ids, wt, gt = torch.empty(N, top, dtype=torch.int32, device=dev), torch.empty(N, top, device=dev), torch.empty(N, device=dev)
+        route = lambda: kernels.moe_route(logits[:, :E], None, ids, wt, None, E, top, 1, 1, 1.0, 1e-20)
+        add("router: sigmoid scores, 4 of 16", "router: sigmoid scores, 4 of 16 from 2 of 4 groups, a gate", timed(route),
+            timed(lambda: kernels.moe_route(logits, None, ids, wt, gt, E, top, 4, 2, 2.5, 1e-20, gate_col=E)), N * (E * 4 + top * 8), N * (E * 4 + top * 8 + 4))
+        route()
+        up, gate_up, down = ((rnd(E, *s_) * 0.1).to(bf) for s_ in ((ffe, W), (2 * ffe, W), (W, ffe)))
+        hid = torch.empty(N * top, ffe, device=dev, dtype=bf)
+        for n, _, what in both:
+            pairs_ = torch.empty(n * top, dtype=torch.int32, device=dev)
+            tiles = torch.empty(kernels.moe_max_tiles(n * top, E), 4, dtype=torch.int32, device=dev)
+            kernels.moe_sort(ids[:n], E, pairs_, tiles)
+            chosen = len(set(ids[:n].flatten().tolist()))
+            kw = (lambda k_: dict(flops=2 * n * top * ffe * W, flops_like=2 * n * top * k_ * ffe * W)) if n == N \
+                else (lambda k_: dict(nbytes=chosen * ffe * W * 2, nbytes_like=chosen * k_ * ffe * W * 2))
+            add(f"experts' first product with the square of relu, {what}", "experts' gate/up product with SiLU",
+                timed(lambda: kernels.moe_gemm(x[:n], up, hid[:n * top], pairs_, tiles, top, gather=True, scatter=False, epi="relu2")),
+                timed(lambda: kernels.moe_gemm(x[:n], gate_up, hid[:n * top], pairs_, tiles, top, gather=True, scatter=False, epi="silu_mul")), **kw(2))
+            add(f"experts' second product, {what}", "the same",
+                *[timed(lambda: kernels.moe_gemm(hid[:n * top], down, pairs_y[:n * top], pairs_, tiles, top, gather=False, scatter=True))] * 2, **kw(1))
+        lgt, like_x = rnd(B, FAMILY_VOCAB), rnd(B, FAMILY_VOCAB)
+        add("cap of the logits, decode b8", "a float32 scale in place", timed(lambda: kernels.softcap(lgt, 30.0)), timed(lambda: kernels.scale_rows(like_x, 1.0)),
+            B * FAMILY_VOCAB * 8)
+        return rows
+
     sizes = {}
-    if args.family in ("kipezen", "fovunex", "gavatar", "nurilorn") and args.family_step:
+    if args.family in ("kipezen", "fovunex", "gavatar", "nurilorn", "nurasun") and args.family_step:
         # one step launched kernel by kernel (no graphs) between cudaProfilerStart / Stop, for a launch list:
         #   ncu --metrics gpu__time_duration.sum --clock-control none --profile-from-start off --csv --log-file L \
         #       python bench.py --family kipezen --family-sizes w2048 --family-step decode
@@ -1405,7 +1590,7 @@ def run_family(args):
         from inf_engine_b200.weights import write_random_model
         size = (args.family_sizes or "w2048").split(",")[0]
         kpz, _ = {"kipezen": _kipezen_configs, "fovunex": _fovunex_configs, "gavatar": _gavatar_configs,
-                  "nurilorn": _nurilorn_configs}[args.family](size)
+                  "nurilorn": _nurilorn_configs, "nurasun": _nurasun_configs}[args.family](size)
         with tempfile.TemporaryDirectory() as tmp:
             write_random_model(kpz, args.seed, tmp)
             r = ModelRunner.from_dir(tmp, dtype="bfloat16", page_size=PAGE, n_pages=(args.batch + 1) * POOL_CONTEXT // PAGE,
@@ -1432,6 +1617,24 @@ def run_family(args):
         torch.cuda.cudart().cudaProfilerStop()
         clocks.stop()
         print(json.dumps({"impl": "ours", "family": args.family, "step": args.family_step, "size": size, "launches": kernels.LAUNCHES}))
+        return 0
+    if args.family == "nurasun":
+        for size in (args.family_sizes.split(",") if args.family_sizes else list(FAMILY_SIZES)):
+            sun, fvx = _nurasun_configs(size)
+            rec = {"nurasun": model_numbers_of(sun, args.batch), "fovunex": model_numbers_of(fvx, args.batch)}
+            rec["kernels"] = nurasun_kernel_table(size)
+            sizes[size] = rec
+        clocks.stop()
+        print(json.dumps({"impl": "ours", "family": "nurasun", "dtype": "bf16", "n_gpus": 1, "steps": args.steps,
+                          "warmup": max(args.warmup, 3),
+                          "data": "synthetic: seeded random weights, uniform random prompt ids",
+                          "config": {"layers": FAMILY_LAYERS, "pattern": "attention in chunks, latent, latent reading it, attention; dense and routed feed-forwards in turn",
+                                     "beside": "two-map attention in chunks, latent, latent, two-map attention (Fovunex), dense feed-forwards",
+                                     "vocab": FAMILY_VOCAB, "head_dim": FAMILY_HD, "prompt": PROMPT_LEN, "decode_batch": args.batch,
+                                     "page_size": PAGE, "chunk": FOVUNEX_CHUNK, "kv_rank": FOVUNEX_RANK, "experts": "16, 4 a token, a shared one",
+                                     "l2": "a 256 MB buffer is written before every timed kernel; model steps stream their weights",
+                                     "sizes": FAMILY_SIZES},
+                          "peaks": pk, "sizes": sizes, "clocks": clocks.summary(t_all0, time.perf_counter())}))
         return 0
     if args.family == "nurilorn":
         for size in (args.family_sizes.split(",") if args.family_sizes else list(FAMILY_SIZES)):
@@ -1703,11 +1906,11 @@ def main():
     ap.add_argument("--no-workloads", action="store_true",
                     help="leave out the two continuous-batching workloads at the other models' sizes")
     ap.add_argument("--family", default=None, metavar="NAME",
-                    help="instead of the default workload: prefill and decode of another model family (barerax, kipezen, fovunex, gavatar, nurilorn) at sizes like "
+                    help="instead of the default workload: prefill and decode of another model family (barerax, kipezen, fovunex, gavatar, nurilorn, nurasun) at sizes like "
                          "a real model's layers, beside the closest earlier model of equal size, and its kernels beside the like ones")
     ap.add_argument("--family-sizes", default=None, help="comma-separated subset of the family's sizes (w1024,w2048)")
     ap.add_argument("--family-step", default=None, choices=["decode", "prefill"],
-                    help="with --family kipezen, fovunex, gavatar or nurilorn: run one such step kernel by kernel between cudaProfilerStart/Stop (for a launch list) and exit")
+                    help="with --family kipezen, fovunex, gavatar, nurilorn or nurasun: run one such step kernel by kernel between cudaProfilerStart/Stop (for a launch list) and exit")
     ap.add_argument("--workload", default=None, metavar="N:MIN:MAX:NEW[:TEMP]",
                     help="instead of the step measurements: N requests through Engine.run_offline (continuous batching)")
     args = ap.parse_args()

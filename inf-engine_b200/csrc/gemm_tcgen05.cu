@@ -6,6 +6,13 @@
 //   SILU_MUL     weight rows alternate gate_j, up_j; C[M, N/2] = silu(gate_j) * up_j   (engine/llama_mlp.py:30-32)
 //   RESIDUAL     C float32 [M, N] += product                                            (engine/llama_block.py:54,62)
 //   RELU2        C bf16, max(product, 0)^2: the first product of a feed-forward without a gate
+//   F32          C float32 [M, N]
+//
+// The grouped form multiplies the rows of a mixture's experts, sorted by expert, each by its own expert's weights: a table of
+// row tiles (expert, first row, rows), none of which spans two experts, stands in for the even cut of M; a tile's rows beyond
+// its own belong to the next expert (or are zero beyond the matrix) and are dropped by the epilogue, which may put each row
+// in a place of its own (the pair's).
+//
 // The plain product is what the reference leaves to a library; the fused epilogues save the round trip of
 // the [M, 2*intermediate] gate/up matrix and of the projections' outputs through HBM.
 //
@@ -20,7 +27,7 @@
 
 namespace {
 
-enum { TC_EPI_BF16 = 0, TC_EPI_SILU_MUL = 3, TC_EPI_RESIDUAL = 2, TC_EPI_RELU2 = 5 };
+enum { TC_EPI_BF16 = 0, TC_EPI_SILU_MUL = 3, TC_EPI_RESIDUAL = 2, TC_EPI_RELU2 = 5, TC_EPI_F32 = 1 };
 
 constexpr int BM = 128;
 constexpr int BK = 64;               // one 128-byte swizzle atom of bfloat16
@@ -43,6 +50,11 @@ struct TcParams {
   // g' sigmoid(act_alpha g' + act_cubic g'^3) (u' + up_offset)
   int act_general;
   float act_alpha, act_limit, up_offset, act_cubic;
+  // grouped form: tiles [max_tiles, 4] = (expert, first row, rows, -), the number of tiles in word 3 of the first; output row
+  // of a sorted row: `place`[row], or the row itself when that is null
+  const int* tiles;
+  const int* place;
+  int max_tiles;
 };
 
 // the gated activation of the SILU_MUL epilogue: silu(g) * u, or with the options above
@@ -115,7 +127,7 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
 
 // one row's 32 accumulator columns n .. n+31 through the epilogue p.epi
 __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, int m, int n, const uint32_t (&r)[32]) {
-  if (m < p.M && n < p.N) {
+  if (m >= 0 && m < p.M && n < p.N) {
     if (p.epi == TC_EPI_BF16 || p.epi == TC_EPI_RELU2) {
       const bool sq = p.epi == TC_EPI_RELU2;
       bf16* dst = (bf16*)p.C + (size_t)m * p.ldc + n;
@@ -158,6 +170,11 @@ __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, int m, int 
           }
         }
       }
+    } else if (p.epi == TC_EPI_F32) {
+      float* dst = (float*)p.C + (size_t)m * p.ldc + n;
+#pragma unroll
+      for (int j = 0; j < 32; ++j)
+        if (n + j < p.N) dst[j] = __uint_as_float(r[j]);
     } else {
       float* dst = (float*)p.C + (size_t)m * p.ldc + n;
       if (n + 32 <= p.N && (((uintptr_t)dst) & 15) == 0) {
@@ -224,15 +241,18 @@ __device__ __forceinline__ void tc_stage_row(const TcParams& p, unsigned char* s
 }
 
 // the warp's tile (rows row0 .. row0 + 31, 128 bytes from byte col_byte0 of each output row) to memory, four rows
-// per instruction; the residual epilogue adds into what is there
-__device__ __forceinline__ void tc_flush(const TcParams& p, const unsigned char* stage, int lane, int row0, size_t col_byte0) {
-  const size_t pitch = (size_t)p.ldc * (p.epi == TC_EPI_RESIDUAL ? 4 : 2);
+// per instruction; the residual epilogue adds into what is there.  GROUPED: this lane's output row is my_row (negative: none)
+template <bool GROUPED>
+__device__ __forceinline__ void tc_flush(const TcParams& p, const unsigned char* stage, int lane, int row0, int my_row,
+                                         size_t col_byte0) {
+  const size_t pitch = (size_t)p.ldc * ((p.epi == TC_EPI_RESIDUAL || p.epi == TC_EPI_F32) ? 4 : 2);
   const int u = lane & 7;
 #pragma unroll
   for (int it = 0; it < 8; ++it) {
-    const int r = it * 4 + (lane >> 3), row = row0 + r;
+    const int r = it * 4 + (lane >> 3);
+    const int row = GROUPED ? __shfl_sync(0xffffffffu, my_row, r) : row0 + r;
     const uint4 v = *reinterpret_cast<const uint4*>(stage + r * 128 + ((u ^ (r & 7)) << 4));
-    if (row < p.M) {
+    if (row >= 0 && row < p.M) {
       unsigned char* dst = (unsigned char*)p.C + (size_t)row * pitch + col_byte0 + (u << 4);
       if (p.epi == TC_EPI_RESIDUAL) {
         float4 g = *reinterpret_cast<float4*>(dst);
@@ -248,7 +268,7 @@ __device__ __forceinline__ void tc_flush(const TcParams& p, const unsigned char*
   }
 }
 
-template <int BN>
+template <int BN, bool GROUPED>
 __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                                                                      const __grid_constant__ CUtensorMap map_w,
                                                                      TcParams p) {
@@ -265,9 +285,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __gri
   const uint32_t full0 = saddr(&bars[0]), empty0 = saddr(&bars[8]);
   const uint32_t acc_full0 = saddr(&bars[16]), acc_empty0 = saddr(&bars[18]);
   const int k_blocks = p.K / BK;
-  const int m_tiles = (p.M + BM - 1) / BM, n_tiles = (p.N + BN - 1) / BN;
-  const int total_tiles = m_tiles * n_tiles;   // tile t: rows (t % m_tiles), columns (t / m_tiles): blocks that run
-                                               // side by side share a weight tile, which then comes from HBM once
+  const int n_tiles = (p.N + BN - 1) / BN;
 
   if (tid == 0) {
     failed = 0;
@@ -292,21 +310,26 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __gri
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   const uint32_t tmem_base = tmem_base_slot;
 
-  pdl_wait();   // the activations come from the kernel ahead
+  pdl_wait();   // the activations (and the table of tiles) come from the kernel ahead
+  const int m_tiles = GROUPED ? max(0, min(p.tiles[3], p.max_tiles)) : (p.M + BM - 1) / BM;
+  const int total_tiles = m_tiles * n_tiles;   // tile t: rows (t % m_tiles), columns (t / m_tiles): blocks that run
+                                               // side by side share a weight tile, which then comes from HBM once
 
   if (warp == 0) {
     if (lane == 0) {
       int s = 0;
       uint32_t phase = 0;
       for (int t = blockIdx.x; t < total_tiles && !failed; t += gridDim.x) {
-        const int m0 = (t % m_tiles) * BM, n0 = (t / m_tiles) * BN;
+        const int mt = t % m_tiles, n0 = (t / m_tiles) * BN;
+        const int m0 = GROUPED ? p.tiles[4 * mt + 1] : mt * BM;
+        const int w0 = GROUPED ? p.tiles[4 * mt] * p.N + n0 : n0;      // the expert's own rows of the stacked weights
         for (int kb = 0; kb < k_blocks; ++kb) {
           if (failed || !tc_mbar_wait(empty0 + 8 * s, phase ^ 1)) { atomicExch(&g_tc_error, 1); failed = 1; break; }
           const uint32_t bar = full0 + 8 * s;
           tc_mbar_expect_tx(bar, STAGE_BYTES);
           const uint32_t a_dst = ring + s * STAGE_BYTES, w_dst = a_dst + A_BYTES;
           tma_load_2d(a_dst, &map_a, kb * BK, m0, bar);
-          tma_load_2d(w_dst, &map_w, kb * BK, n0, bar);
+          tma_load_2d(w_dst, &map_w, kb * BK, w0, bar);
           if (++s == p.n_stages) { s = 0; phase ^= 1; }
         }
       }
@@ -350,8 +373,12 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __gri
     for (int t = blockIdx.x; t < total_tiles; t += gridDim.x, ++it) {
       const int buf = it & 1;
       const uint32_t acc_phase = (uint32_t)(it >> 1) & 1u;
-      const int m0 = (t % m_tiles) * BM, n0 = (t / m_tiles) * BN;
-      const int m = m0 + quarter * 32 + lane;
+      const int mt = t % m_tiles, n0 = (t / m_tiles) * BN;
+      int m = mt * BM + quarter * 32 + lane;
+      if (GROUPED) {
+        const int r = quarter * 32 + lane, src = p.tiles[4 * mt + 1] + r;
+        m = r < p.tiles[4 * mt + 2] ? (p.place != nullptr ? p.place[src] : src) : -1;
+      }
       bool ok = !failed && tc_mbar_wait(acc_full0 + 8 * buf, acc_phase);
       if (!ok && lane == 0) { atomicExch(&g_tc_error, 3); failed = 1; }
       ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0 && !failed;
@@ -375,7 +402,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __gri
           off += out32;
           if (off == 128) {
             __syncwarp();
-            tc_flush(p, stage, lane, m - lane, (size_t)(n0 + c0 + 32) * (out32 >> 5) - 128);
+            tc_flush<GROUPED>(p, stage, lane, m - lane, m, (size_t)(n0 + c0 + 32) * (out32 >> 5) - 128);
             __syncwarp();
             off = 0;
           }
@@ -424,7 +451,7 @@ static int make_map(CUtensorMap* map, const void* base, int rows, int cols, int 
   return r == CUDA_SUCCESS ? IE_OK : IE_BAD_ALIGN;
 }
 
-template <int BN>
+template <int BN, bool GROUPED>
 static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mw, TcParams p, int n_sms, cudaStream_t stream) {
   const uint32_t stage = (BM + BN) * BK * 2;
   int n_stages = (200 * 1024 - 1024) / stage;
@@ -433,13 +460,13 @@ static int launch_tc(const CUtensorMap& ma, const CUtensorMap& mw, TcParams p, i
   const size_t smem = (size_t)n_stages * stage + 1024 + 4 * TC_STAGE_BYTES;
   static bool attr = false;
   if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     attr = true;
   }
-  const int tiles = ((p.M + BM - 1) / BM) * ((p.N + BN - 1) / BN);
+  const int tiles = (GROUPED ? p.max_tiles : (p.M + BM - 1) / BM) * ((p.N + BN - 1) / BN);
   const int grid = tiles < n_sms ? tiles : n_sms;
-  return launch_k(gemm_tcgen05_kernel<BN>, grid, TC_THREADS, smem, stream, ma, mw, p);
+  return launch_k(gemm_tcgen05_kernel<BN, GROUPED>, grid, TC_THREADS, smem, stream, ma, mw, p);
 }
 
 }  // namespace
@@ -481,7 +508,37 @@ extern "C" int ie_gemm_tcgen05_act(const void* A, const void* W, void* C, int M,
   p.act_general = act_general; p.act_alpha = act_alpha; p.act_limit = act_limit; p.up_offset = up_offset;
   p.act_cubic = act_cubic;
   p.staged = (((uintptr_t)C & 15) == 0 && ((size_t)ldc * (epi == TC_EPI_RESIDUAL ? 4 : 2)) % 16 == 0) ? 1 : 0;
-  return bn == 256 ? launch_tc<256>(ma, mw, p, n_sms, stream) : launch_tc<128>(ma, mw, p, n_sms, stream);
+  p.tiles = nullptr; p.place = nullptr; p.max_tiles = 0;
+  return bn == 256 ? launch_tc<256, false>(ma, mw, p, n_sms, stream) : launch_tc<128, false>(ma, mw, p, n_sms, stream);
+}
+
+extern "C" int ie_gemm_tcgen05_tile_rows() { return BM; }
+
+// The grouped form: A [n_rows, K] sorted by expert, W [experts, N, K]; epi 1 (float32), 3 or 5.  `place` (optional) names the
+// output row of every sorted row; C has n_rows rows.
+extern "C" int ie_gemm_tcgen05_grouped(const void* A, const void* W, void* C, const int* tiles, const int* place, int max_tiles,
+                                       int n_rows, int experts, int N, int K, int lda, int ldc, int epi, int bn, int n_sms,
+                                       float act_alpha, float act_limit, float up_offset, float act_cubic,
+                                       cudaStream_t stream) {
+  if (n_sms <= 0 || experts <= 0) return IE_BAD_SIZE;
+  if (n_rows <= 0 || N <= 0 || max_tiles <= 0) return IE_OK;
+  if (!ie_gemm_tcgen05_supports(n_rows, N, K, lda, K)) return IE_BAD_SIZE;
+  if ((long long)experts * N > 0x7fffffffLL) return IE_BAD_SIZE;
+  if (((uintptr_t)A | (uintptr_t)W) & 15) return IE_BAD_ALIGN;
+  if (epi != TC_EPI_F32 && epi != TC_EPI_SILU_MUL && epi != TC_EPI_RELU2) return IE_BAD_DTYPE;
+  if (epi == TC_EPI_SILU_MUL && (N & 1)) return IE_BAD_SIZE;
+  if (bn != 128 && bn != 256) return IE_BAD_SIZE;
+  CUtensorMap ma, mw;
+  int rc = make_map(&ma, A, n_rows, K, lda, BM);
+  if (rc) return rc;
+  rc = make_map(&mw, W, experts * N, K, K, bn);
+  if (rc) return rc;
+  TcParams p;
+  p.C = C; p.M = n_rows; p.N = N; p.K = K; p.ldc = ldc; p.epi = epi; p.n_stages = 0;
+  p.act_general = 1; p.act_alpha = act_alpha; p.act_limit = act_limit; p.up_offset = up_offset; p.act_cubic = act_cubic;
+  p.tiles = tiles; p.place = place; p.max_tiles = max_tiles;
+  p.staged = (((uintptr_t)C & 15) == 0 && ((size_t)ldc * (epi == TC_EPI_F32 ? 4 : 2)) % 16 == 0) ? 1 : 0;
+  return bn == 256 ? launch_tc<256, true>(ma, mw, p, n_sms, stream) : launch_tc<128, true>(ma, mw, p, n_sms, stream);
 }
 
 extern "C" int ie_gemm_tcgen05(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,

@@ -18,7 +18,8 @@
 // cosines of a block's tokens worked out once and shared by all heads.
 //
 // heads_gemm: a product per head, out[m, h, j] = sum_k x[m, h, k] * w[h, k, j], float32 products summed in ascending k
-// (the same for a row whatever else is in the batch), any of float32 and bfloat16 for x, w and out.
+// (the same for a row whatever else is in the batch), any of float32 and bfloat16 for x, w and out.  A few rows (decode
+// tokens) take a form whose warps split k and whose partial sums are added in warp order.
 //
 // diff_combine: two attention maps of a head that share their values become one output:
 //   o = a1 - lambda * a2;  o <- o / sqrt(mean(o^2) + eps) * out_mult * sigmoid(gate)      (gate optional)
@@ -215,6 +216,39 @@ __global__ void __launch_bounds__(RW_THREADS) rotate_write_kernel(RotateWritePar
   }
 }
 
+// One key row a token whose norm covers all of it, nothing turned, no queries and no values (a compressed vector on its way
+// to the cache): a warp a token.
+#define KR_WARPS 8
+
+template <typename TA, typename TW>
+__global__ void __launch_bounds__(KR_WARPS * 32) key_row_norm_kernel(const TA* __restrict__ k, int k_stride, int hd,
+                                                                     const TW* __restrict__ gain, float eps,
+                                                                     const int* __restrict__ slot_mapping,
+                                                                     TA* __restrict__ kpool, int n_tokens) {
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, n = blockIdx.x * KR_WARPS + (threadIdx.x >> 5);
+  if (n >= n_tokens) return;
+  const int slot = IE_SLOT(slot_mapping[n]);
+  if (slot < 0) return;
+  const TA* row = k + (size_t)n * k_stride;
+  float v[8];                            // hd up to 256
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int d = lane + 32 * i;
+    v[i] = d < hd ? to_f32(row[d]) : 0.f;
+    ss = fmaf(v[i], v[i], ss);
+  }
+  const float r = sqrtf(warp_sum(ss) / (float)hd + eps);
+  TA* dst = kpool + (size_t)slot * hd;   // one head: the page and the place in it make one row index
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int d = lane + 32 * i;
+    if (d < hd) dst[d] = from_f32<TA>(v[i] / r * to_f32(gain[d]));
+  }
+}
+
 // tied: the key rows with their bias, before norm and rotation, are also the values (v is then ignored; the pool has the
 // keys' heads and head size)
 extern "C" int ie_head_prepare(void* q, int q_stride, int q_heads, int q_hd, int q_norm_dims, int q_rot_off,
@@ -246,6 +280,19 @@ extern "C" int ie_head_prepare(void* q, int q_stride, int q_heads, int q_hd, int
     const size_t cs_bytes = sizeof(float2) * p.tokens_a_block * (size_t)(rot >> 1);
     if (w_dtype == IE_F32) return launch_k(rotate_write_kernel<float>, blocks, RW_THREADS, cs_bytes, stream, p);
     if (w_dtype == IE_BF16) return launch_k(rotate_write_kernel<bf16>, blocks, RW_THREADS, cs_bytes, stream, p);
+    return IE_BAD_DTYPE;
+  }
+  if (q_heads == 0 && k_heads == 1 && k_gain != nullptr && k_bias == nullptr && k_norm_dims == k_hd && k_hd <= 256 && rot == 0 &&
+      v == nullptr && !tied && kpool != nullptr && slot_mapping != nullptr) {
+    const int blocks = (n_tokens + KR_WARPS - 1) / KR_WARPS;
+#define KR_GO(TA, TW)                                                                                                    \
+  return launch_k(key_row_norm_kernel<TA, TW>, blocks, KR_WARPS * 32, 0, stream, (const TA*)k, k_stride, k_hd, (const TW*)k_gain, \
+                  eps, slot_mapping, (TA*)kpool, n_tokens)
+    if (act_dtype == IE_F32 && w_dtype == IE_F32) KR_GO(float, float);
+    if (act_dtype == IE_F32 && w_dtype == IE_BF16) KR_GO(float, bf16);
+    if (act_dtype == IE_BF16 && w_dtype == IE_F32) KR_GO(bf16, float);
+    if (act_dtype == IE_BF16 && w_dtype == IE_BF16) KR_GO(bf16, bf16);
+#undef KR_GO
     return IE_BAD_DTYPE;
   }
   const size_t smem = sizeof(float) * ((size_t)q_heads * q_hd + (size_t)k_heads * k_hd);
@@ -314,10 +361,104 @@ __global__ void __launch_bounds__(HG_THREADS) heads_gemm_kernel(const TX* __rest
   }
 }
 
+// Few rows: block (j block, head, row group) takes 64 columns of a head (two a lane) and HG_ROWS rows; its warps take
+// equal runs of k, so that every weight of the block is on its way at once, and their sums are added in warp order.
+#define HS_WARPS 8
+
+template <typename T> __device__ __forceinline__ float2 load2(const T* p);
+template <> __device__ __forceinline__ float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> __device__ __forceinline__ float2 load2<bf16>(const bf16* p) {
+  return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+
+template <typename TX, typename TW, typename TO>
+__global__ void __launch_bounds__(HS_WARPS * 32) heads_gemm_few_kernel(const TX* __restrict__ x, int x_stride, int x_head,
+                                                                       const TW* __restrict__ w, TO* __restrict__ out,
+                                                                       int o_stride, int o_head, int M, int K, int N) {
+  extern __shared__ float xs[];          // [HG_ROWS][K], then [HS_WARPS][HG_ROWS][64]
+  float* part = xs + (size_t)HG_ROWS * K;
+  const int h = blockIdx.y, m0 = blockIdx.z * HG_ROWS, rows = min(HG_ROWS, M - m0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j = blockIdx.x * 64 + lane * 2;
+  const int per = (K + HS_WARPS - 1) / HS_WARPS, k_lo = min(K, warp * per), k_hi = min(K, k_lo + per);
+  const TW* wh = w + (size_t)h * K * N + j;
+  constexpr int AHEAD = 16;              // weights fetched before the kernel ahead has finished: they do not depend on it
+  float2 first[AHEAD];
+#pragma unroll
+  for (int u = 0; u < AHEAD; ++u)
+    first[u] = (j < N && k_lo + u < k_hi) ? load2<TW>(wh + (size_t)(k_lo + u) * N) : make_float2(0.f, 0.f);
+  pdl_trigger();
+  pdl_wait();
+  for (int i = threadIdx.x; i < HG_ROWS * K; i += HS_WARPS * 32) {
+    const int r = i / K, k = i - r * K;
+    xs[i] = r < rows ? to_f32(x[(size_t)(m0 + r) * x_stride + h * x_head + k]) : 0.f;
+  }
+  __syncthreads();
+  float2 acc[HG_ROWS];
+#pragma unroll
+  for (int r = 0; r < HG_ROWS; ++r) acc[r] = make_float2(0.f, 0.f);
+  for (int k0 = k_lo; k0 < k_hi; k0 += AHEAD) {
+    float2 next[AHEAD];
+    if (k0 + AHEAD < k_hi) {
+#pragma unroll
+      for (int u = 0; u < AHEAD; ++u) {
+        const int k = k0 + AHEAD + u;
+        next[u] = (j < N && k < k_hi) ? load2<TW>(wh + (size_t)k * N) : make_float2(0.f, 0.f);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      if (k0 + u >= k_hi) break;
+#pragma unroll
+      for (int r = 0; r < HG_ROWS; ++r) {
+        const float v = xs[r * K + k0 + u];
+        acc[r].x = fmaf(v, first[u].x, acc[r].x);
+        acc[r].y = fmaf(v, first[u].y, acc[r].y);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) first[u] = next[u];
+  }
+#pragma unroll
+  for (int r = 0; r < HG_ROWS; ++r)
+    *reinterpret_cast<float2*>(part + ((size_t)warp * HG_ROWS + r) * 64 + lane * 2) = acc[r];
+  __syncthreads();
+  for (int i = threadIdx.x; i < rows * 64; i += HS_WARPS * 32) {
+    const int r = i >> 6, c = i & 63, col = blockIdx.x * 64 + c;
+    if (col >= N) continue;
+    float s = 0.f;
+#pragma unroll
+    for (int v = 0; v < HS_WARPS; ++v) s += part[((size_t)v * HG_ROWS + r) * 64 + c];
+    out[(size_t)(m0 + r) * o_stride + h * o_head + col] = from_f32<TO>(s);
+  }
+}
+
+template <typename TX, typename TW, typename TO>
+static int launch_heads_few(const void* x, int x_stride, int x_head, const void* w, void* out, int o_stride, int o_head, int M,
+                            int H, int K, int N, cudaStream_t stream) {
+  const size_t smem = sizeof(float) * ((size_t)HG_ROWS * K + (size_t)HS_WARPS * HG_ROWS * 64);
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(heads_gemm_few_kernel<TX, TW, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  dim3 grid((N + 63) / 64, H, (M + HG_ROWS - 1) / HG_ROWS);
+  return launch_k(heads_gemm_few_kernel<TX, TW, TO>, grid, HS_WARPS * 32, smem, stream, (const TX*)x, x_stride, x_head,
+                  (const TW*)w, (TO*)out, o_stride, o_head, M, K, N);
+}
+
 extern "C" int ie_heads_gemm(const void* x, int x_dtype, int x_stride, int x_head, const void* w, int w_dtype, void* out,
                              int o_dtype, int o_stride, int o_head, int M, int H, int K, int N, cudaStream_t stream) {
   if (M <= 0 || H <= 0 || N <= 0) return IE_OK;
   if (K <= 0 || H > 65535) return IE_BAD_SIZE;
+  if (M <= 16 && (N & 1) == 0 && ((uintptr_t)w & 7) == 0 && (size_t)HG_ROWS * K * sizeof(float) <= 64 * 1024) {
+#define HS_GO(TX, TW, TO) return launch_heads_few<TX, TW, TO>(x, x_stride, x_head, w, out, o_stride, o_head, M, H, K, N, stream)
+    if (x_dtype == IE_F32 && w_dtype == IE_F32 && o_dtype == IE_F32) HS_GO(float, float, float);
+    if (x_dtype == IE_F32 && w_dtype == IE_BF16 && o_dtype == IE_F32) HS_GO(float, bf16, float);
+    if (x_dtype == IE_BF16 && w_dtype == IE_BF16 && o_dtype == IE_BF16) HS_GO(bf16, bf16, bf16);
+    if (x_dtype == IE_BF16 && w_dtype == IE_F32 && o_dtype == IE_BF16) HS_GO(bf16, float, bf16);
+#undef HS_GO
+    return IE_BAD_DTYPE;
+  }
   // narrow outputs and enough rows: two or four row groups a block (a row's sum is the same whichever group forms it)
   int groups = N <= 32 ? 4 : (N <= 64 ? 2 : 1);
   while (groups > 1 && (M < groups * HG_ROWS || sizeof(float) * groups * HG_ROWS * (size_t)K > 96 * 1024)) groups >>= 1;

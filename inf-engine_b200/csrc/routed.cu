@@ -142,7 +142,7 @@ extern "C" int ie_moe_route(const float* logits, int ld, const void* correction,
 // ------------------------------------------------------------------ sort
 // One block.  sorted[pos] = pair index (token * top + choice) with the pairs of expert 0 first, then expert 1, ...;
 // tiles[4 * i .. 4 * i + 3] = (expert, first position, rows, 0) for every tile of at most `tile_rows` rows; tiles
-// beyond the last carry rows = 0.  The order of an expert's pairs among themselves is whatever the atomics give:
+// beyond the last carry rows = 0, and word 3 of the first one holds their number.  The order of an expert's pairs among themselves is whatever the atomics give:
 // a pair's result does not depend on its place.
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int n_experts, int tile_rows, int* __restrict__ sorted,
@@ -172,7 +172,9 @@ moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int n_experts, int til
       }
       pos += count[e];
     }
+    const int n_tiles = nt;
     for (; nt < max_tiles; ++nt) tiles[4 * nt] = tiles[4 * nt + 1] = tiles[4 * nt + 2] = tiles[4 * nt + 3] = 0;
+    tiles[3] = n_tiles;
   }
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
@@ -187,6 +189,30 @@ extern "C" int ie_moe_sort(const int* ids, int n_pairs, int n_experts, int tile_
   if (n_experts <= 0 || tile_rows <= 0 || 3 * (size_t)n_experts * sizeof(int) > 47 * 1024) return IE_BAD_SIZE;
   return launch_k(moe_sort_kernel, 1, 1024, 3 * (size_t)n_experts * sizeof(int), stream, ids, n_pairs, n_experts,
                   tile_rows, sorted, tiles, max_tiles);
+}
+
+// ------------------------------------------------------------------ rows in sorted order
+// out[pos] = x[sorted[pos] / top] in 16-byte pieces: what the grouped product on tcgen05 reads, whose rows must lie in a row
+__global__ void moe_gather_kernel(const bf16* __restrict__ x, int x_stride, bf16* __restrict__ out, const int* __restrict__ sorted,
+                                  int top, int pieces, size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const size_t pos = i / pieces;
+  const int c = (int)(i - pos * pieces) * 8;
+  *reinterpret_cast<uint4*>(out + pos * pieces * 8 + c) =
+      *reinterpret_cast<const uint4*>(x + (size_t)(sorted[pos] / top) * x_stride + c);
+}
+
+extern "C" int ie_moe_gather(const void* x, int x_stride, void* out, const int* sorted, int top, int n_pairs, int d,
+                             cudaStream_t stream) {
+  if (n_pairs <= 0) return IE_OK;
+  if (top <= 0 || d <= 0 || d % 8 || x_stride % 8) return IE_BAD_SIZE;
+  if (((uintptr_t)x | (uintptr_t)out) & 15) return IE_BAD_ALIGN;
+  const size_t total = (size_t)n_pairs * (d / 8);
+  return launch_k(moe_gather_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, (const bf16*)x, x_stride, (bf16*)out, sorted,
+                  top, d / 8, total);
 }
 
 // ------------------------------------------------------------------ grouped product
@@ -429,18 +455,118 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* 
   }
 }
 
+// ---- the same product for a few tokens (decode steps), bound by reading the chosen experts' weights once: a block takes 8
+// weight rows of one tile's expert; its eight warps split K in chunks of 32 and a lane loads 16 bytes of a weight row straight
+// into the B fragments of two MMAs (k is permuted inside a chunk in the same way for A and W, which a sum allows), so that up
+// to ST_PREF such loads a lane are on their way; the warps' partial sums are added in warp order.  Tiles of more than 16 rows
+// walk their weights again for every 16.
+#define ST_WARPS 8
+#define ST_PREF 8
+
+__device__ __forceinline__ uint4 st_weights(const bf16* p) {
+  uint4 v;
+  uint64_t pol;
+  asm volatile("createpolicy.fractional.L2::evict_first.b64 %0, 1.0;" : "=l"(pol));
+  asm volatile("ld.global.nc.L1::no_allocate.L2::cache_hint.v4.u32 {%0,%1,%2,%3}, [%4], %5;"
+               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p), "l"(pol));
+  return v;
+}
+
+template <typename TC>
+__global__ void __launch_bounds__(ST_WARPS * 32)
+moe_gemm_stream_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* __restrict__ C,
+                       const int* __restrict__ sorted, const int* __restrict__ tiles, int N, int K, int lda, int ldc,
+                       long long w_expert_stride, int top, int gather, int scatter, int epi, GluAct act) {
+  pdl_trigger();
+  pdl_wait();                                               // which expert a tile belongs to comes from the kernel ahead
+  __shared__ float red[ST_WARPS][4][32];
+  const int tile = blockIdx.y;
+  const int rows = tiles[4 * tile + 2];
+  if (rows <= 0) return;
+  const int expert = tiles[4 * tile], pos0 = tiles[4 * tile + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int n0 = blockIdx.x * 8;
+  const bool w_in = n0 + g < N;
+  const bf16* wrow = W + (size_t)expert * w_expert_stride + (size_t)(w_in ? n0 + g : 0) * K;
+  const int n_chunks = (K + 31) >> 5;
+  const int c_lo = (int)((long long)n_chunks * warp / ST_WARPS), c_hi = (int)((long long)n_chunks * (warp + 1) / ST_WARPS);
+  for (int r0 = 0; r0 < rows; r0 += 16) {
+    const bf16* arow[2];
+    bool a_in[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = r0 + g + 8 * h;
+      a_in[h] = r < rows;
+      const int row = !a_in[h] ? 0 : (gather ? sorted[pos0 + r] / top : pos0 + r);
+      arow[h] = A + (size_t)row * lda;
+    }
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int base = c_lo; base < c_hi; base += ST_PREF) {
+      uint4 w[ST_PREF], a[ST_PREF][2];
+#pragma unroll
+      for (int j = 0; j < ST_PREF; ++j) {
+        const int k = ((base + j) << 5) + t * 8;
+        const bool in = base + j < c_hi && k < K;
+        w[j] = (in && w_in) ? st_weights(wrow + k) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+          a[j][h] = (in && a_in[h]) ? *reinterpret_cast<const uint4*>(arow[h] + k) : make_uint4(0u, 0u, 0u, 0u);
+      }
+#pragma unroll
+      for (int j = 0; j < ST_PREF; ++j) {
+        const uint32_t lo[4] = {a[j][0].x, a[j][1].x, a[j][0].y, a[j][1].y}, hi[4] = {a[j][0].z, a[j][1].z, a[j][0].w, a[j][1].w};
+        mm_mma(acc, lo, w[j].x, w[j].y);
+        mm_mma(acc, hi, w[j].z, w[j].w);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) red[warp][e][lane] = acc[e];
+    __syncthreads();
+    if (threadIdx.x < 64) {
+      // thread (half h, lane): row g + 8 h, columns 2 t and 2 t + 1
+      const int h = threadIdx.x >> 5;
+      float x0 = 0.f, x1 = 0.f;
+#pragma unroll
+      for (int v = 0; v < ST_WARPS; ++v) {
+        x0 += red[v][2 * h][lane];
+        x1 += red[v][2 * h + 1][lane];
+      }
+      const int r = r0 + g + 8 * h, n = n0 + t * 2;
+      if (r < rows && n < N) {
+        const size_t cr = scatter ? sorted[pos0 + r] : pos0 + r;
+        if (epi == 1) {
+          if (n + 1 < N) C[cr * ldc + (n >> 1)] = from_f32<TC>(glu(act, x0, x1));
+        } else {
+          C[cr * ldc + n] = from_f32<TC>(plain_act(epi, x0));
+          if (n + 1 < N) C[cr * ldc + n + 1] = from_f32<TC>(plain_act(epi, x1));
+        }
+      }
+    }
+    __syncthreads();
+  }
+}
+
 extern "C" int ie_moe_tile_rows() { return MG_BM; }
 
+// few: the step has few tokens (no expert gets more rows than about 16): bfloat16 operands take the weight-streaming form
 extern "C" int ie_moe_gemm(const void* A, int a_dtype, const void* W, int w_dtype, void* C, int c_dtype,
                            const int* sorted, const int* tiles, int max_tiles, int N, int K, int lda, int ldc,
                            long long w_expert_stride, int top, int gather, int scatter, int epi, float alpha, float limit,
-                           float up_offset, float cubic, cudaStream_t stream) {
+                           float up_offset, float cubic, int few, cudaStream_t stream) {
   const GluAct act{alpha, limit, up_offset, cubic};
   if (max_tiles <= 0 || N <= 0) return IE_OK;
   if (K <= 0 || top <= 0 || (epi == 1 && (N & 1))) return IE_BAD_SIZE;
   if (a_dtype == IE_BF16 && w_dtype == IE_BF16 && K % 8 == 0 && lda % 8 == 0 && w_expert_stride % 8 == 0 &&
       (((uintptr_t)A | (uintptr_t)W) & 15) == 0) {
     static_assert(MM_BM == MG_BM, "both kernels walk the same tiles");
+    if (few) {
+      dim3 few_grid((N + 7) / 8, max_tiles);
+      if (c_dtype == IE_BF16)
+        return launch_k(moe_gemm_stream_kernel<bf16>, few_grid, ST_WARPS * 32, 0, stream, (const bf16*)A, (const bf16*)W, (bf16*)C,
+                        sorted, tiles, N, K, lda, ldc, w_expert_stride, top, gather, scatter, epi, act);
+      return launch_k(moe_gemm_stream_kernel<float>, few_grid, ST_WARPS * 32, 0, stream, (const bf16*)A, (const bf16*)W, (float*)C,
+                      sorted, tiles, N, K, lda, ldc, w_expert_stride, top, gather, scatter, epi, act);
+    }
     dim3 grid((N + MM_BN - 1) / MM_BN, max_tiles);
     if (c_dtype == IE_BF16)
       return launch_k(moe_gemm_mma_kernel<bf16>, grid, MM_THREADS, 0, stream, (const bf16*)A, (const bf16*)W, (bf16*)C,

@@ -73,9 +73,9 @@ class StepContext:
             for r, q_len in enumerate(self.host["q_lens"]):
                 if q_len * group <= more_than:
                     continue
-                for p in range(0, q_len * group, rows):
-                    req.append(r)
-                    pair0.append(p)
+                tiles = range(0, q_len * group, rows)
+                req.extend([r] * len(tiles))
+                pair0.extend(tiles)
             n = len(req)
             dev = self.rt.staging.upload(np.asarray(req + pair0, dtype=np.int32)) if n else None
             self._work[key] = (dev[:n], dev[n:], n) if n else (None, None, 0)
@@ -126,18 +126,17 @@ def build_context(rt, manager, entries: list[StepEntry]) -> StepContext:
     for g in manager.kv_groups:
         width = max(len(g.tables[e.rid]) for e in entries)
         widths.append(width)
-        slot_map = []
+        slots_of = []
         table = np.full((R, width), -1, dtype=np.int32)
         for r, e in enumerate(entries):
             t = g.tables[e.rid]
             table[r, :len(t)] = t
-            base = ctx_before[r]
-            for p in range(base, base + q_lens[r]):
-                page = t[p // ps]
-                if page < 0:
-                    raise RuntimeError(f"request {e.rid!r}: position {p} lies on a released page")
-                slot_map.append(page * ps + p % ps)
-        parts.append(slot_map)
+            at = np.arange(ctx_before[r], ctx_before[r] + q_lens[r])
+            pages = table[r, at // ps]
+            if pages.min() < 0:
+                raise RuntimeError(f"request {e.rid!r}: position {at[int(pages.argmin())]} lies on a released page")
+            slots_of.append(pages * ps + at % ps)
+        parts.append(np.concatenate(slots_of))
         parts.append(table.reshape(-1))
     flat = np.concatenate([np.asarray(p, dtype=np.int32).reshape(-1) for p in parts])
     dev = rt.staging.upload(flat)

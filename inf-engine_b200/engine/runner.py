@@ -110,9 +110,9 @@ class ModelRunner:
             if new_len > self.spec.max_positions:
                 raise ValueError(f"request {e.rid!r} would reach {new_len} tokens, beyond max_positions="
                                  f"{self.spec.max_positions}")
-            for t in e.tokens:
-                if not 0 <= t < self.spec.vocab_size:
-                    raise ValueError(f"token id {t} of request {e.rid!r} is outside the vocabulary")
+            if e.tokens and not (0 <= min(e.tokens) and max(e.tokens) < self.spec.vocab_size):
+                bad = next(t for t in e.tokens if not 0 <= t < self.spec.vocab_size)
+                raise ValueError(f"token id {bad} of request {e.rid!r} is outside the vocabulary")
         # all or nothing: check first, then take
         need = [0] * len(cache.kv_groups)
         for e in entries:

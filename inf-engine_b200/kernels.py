@@ -99,8 +99,10 @@ def core():
         lib.ie_linear_recurrence.argtypes = [P, I, P, I, P, P, I, P, P, P, I, P, P, I, P, P, I, I, F, F, I, I, P]
         lib.ie_rownorm_rotate_write.argtypes = [P, P, P, I, I, I, P, P, P, P, P, I, F, P, I, P, P, P, P, I, I, I, I, I, I, I, P]
         lib.ie_moe_route.argtypes = [P, I, P, I, P, P, P, I, I, I, I, I, F, F, I, I, I, P]
+        lib.ie_moe_gather.argtypes = [P, I, P, P, I, I, I, P]
+        lib.ie_moe_gather.restype = c_int
         lib.ie_moe_sort.argtypes = [P, I, I, I, P, P, I, P]
-        lib.ie_moe_gemm.argtypes = [P, I, P, I, P, I, P, P, I, I, I, I, I, L, I, I, I, I, F, F, F, F, P]
+        lib.ie_moe_gemm.argtypes = [P, I, P, I, P, I, P, P, I, I, I, I, I, L, I, I, I, I, F, F, F, F, I, P]
         lib.ie_moe_combine.argtypes = [P, P, P, P, I, I, P, I, I, I, P]
         lib.ie_moe_tile_rows.restype = c_int
         lib.ie_head_prepare.argtypes = [P, I, I, I, I, I, P, P, I, I, I, I, I, P, P, P, I, P, I, I, I, I, F, P, I, I, F, P, P, P, P, I, I, I, P]
@@ -764,11 +766,12 @@ def moe_tile_rows() -> int:
     return int(core().ie_moe_tile_rows())
 
 
-def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
+def moe_max_tiles(n_pairs: int, n_experts: int, tile_rows: int | None = None) -> int:
     """An upper bound of the row tiles that ``moe_sort`` makes of ``n_pairs`` pairs (no tile spans two experts)."""
-    return -(-n_pairs // moe_tile_rows()) + min(n_experts, n_pairs)
+    return -(-n_pairs // (tile_rows or moe_tile_rows())) + min(n_experts, n_pairs)
 
 
+MOE_FEW_TOKENS = 16         # up to here the experts' products stream their weights (no expert gets more rows than tokens)
 ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1, "softmax": 2}
 GROUP_SCORES = {"top2_sum": 0, "max": 1}
 
@@ -793,13 +796,15 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, ids: torch.
                                float(weight_eps), int(gate_col), ROUTE_SCORES[score], GROUP_SCORES[group_score], _stream()), f"moe_route(experts={n_experts}, top={top})")
 
 
-def moe_sort(ids: torch.Tensor, n_experts: int, sorted_pairs: torch.Tensor, tiles: torch.Tensor) -> None:
+def moe_sort(ids: torch.Tensor, n_experts: int, sorted_pairs: torch.Tensor, tiles: torch.Tensor, tile_rows: int | None = None) -> None:
     """Order the (token, choice) pairs by expert: ``sorted_pairs`` int32 [n_pairs], ``tiles`` int32 [max_tiles, 4] =
-    (expert, first position, rows, 0)."""
+    (expert, first position, rows, 0), the number of tiles in the last word of the first one.  ``tile_rows``: the most rows
+    of a tile (None: what ``moe_gemm`` takes)."""
     n_pairs = ids.numel()
+    tile_rows = int(tile_rows or moe_tile_rows())
     assert sorted_pairs.dtype is torch.int32 and sorted_pairs.numel() >= n_pairs and tiles.dtype is torch.int32
-    assert tiles.is_contiguous() and tiles.shape[1] == 4 and tiles.shape[0] >= moe_max_tiles(n_pairs, n_experts)
-    _check(core().ie_moe_sort(_ptr(ids), n_pairs, n_experts, moe_tile_rows(), _ptr(sorted_pairs), _ptr(tiles),
+    assert tiles.is_contiguous() and tiles.shape[1] == 4 and tiles.shape[0] >= moe_max_tiles(n_pairs, n_experts, tile_rows)
+    _check(core().ie_moe_sort(_ptr(ids), n_pairs, n_experts, tile_rows, _ptr(sorted_pairs), _ptr(tiles),
                               tiles.shape[0], _stream()), "moe_sort")
 
 
@@ -815,8 +820,17 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, sorted_pairs: to
     _check(core().ie_moe_gemm(_ptr(a), dtype_code(a.dtype), _ptr(w), dtype_code(w.dtype), _ptr(c), dtype_code(c.dtype),
                               _ptr(sorted_pairs), _ptr(tiles), tiles.shape[0], n, k, a.stride(0), c.stride(0), n * k, top,
                               1 if gather else 0, 1 if scatter else 0, {"store": 0, "silu_mul": 1, "relu2": 2}[epi], float(alpha),
-                              float(limit), float(up_offset), float(cubic), _stream()),
+                              float(limit), float(up_offset), float(cubic),
+                              1 if c.shape[0] <= MOE_FEW_TOKENS * top else 0, _stream()),
            f"moe_gemm(n={n}, k={k}, {epi})")
+
+
+def moe_gather(x: torch.Tensor, out: torch.Tensor, sorted_pairs: torch.Tensor, top: int) -> None:
+    """out[pos] = x[sorted_pairs[pos] // top] (bfloat16, rows of a multiple of 8 numbers)."""
+    n, d = out.shape
+    assert x.dtype is torch.bfloat16 and out.dtype is torch.bfloat16 and out.is_contiguous() and x.stride(1) == 1
+    assert sorted_pairs.numel() >= n and x.shape[1] == d
+    _check(core().ie_moe_gather(_ptr(x), x.stride(0), _ptr(out), _ptr(sorted_pairs), top, n, d, _stream()), "moe_gather")
 
 
 def moe_combine(y: torch.Tensor, weights: torch.Tensor, gate: torch.Tensor | None, shared_out: torch.Tensor | None,
@@ -1410,6 +1424,9 @@ def tcgen05_library():
         lib.ie_gemm_tcgen05.restype = c_int
         lib.ie_gemm_tcgen05_act.argtypes = [c_void_p] * 3 + [c_int] * 10 + [c_float] * 4 + [c_void_p]
         lib.ie_gemm_tcgen05_act.restype = c_int
+        lib.ie_gemm_tcgen05_grouped.argtypes = [c_void_p] * 5 + [c_int] * 10 + [c_float] * 4 + [c_void_p]
+        lib.ie_gemm_tcgen05_grouped.restype = c_int
+        lib.ie_gemm_tcgen05_tile_rows.restype = c_int
         lib.ie_gemm_tcgen05_supports.argtypes = [I, I, I, I, I]
         lib.ie_gemm_tcgen05_supports.restype = c_int
         lib.ie_gemm_tcgen05_error.restype = c_int
@@ -1424,6 +1441,28 @@ def gemm_tcgen05_supports(m: int, n: int, k: int, lda: int, ldw: int) -> bool:
 def gemm_tcgen05_error() -> int:
     """Reads and clears the error word that a timed-out wait of the tcgen05 kernel leaves (0: none)."""
     return int(tcgen05_library().ie_gemm_tcgen05_error())
+
+
+def gemm_tcgen05_tile_rows() -> int:
+    return int(tcgen05_library().ie_gemm_tcgen05_tile_rows())
+
+
+def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, tiles: torch.Tensor, place: torch.Tensor | None,
+                         epi: str, act: tuple | None = None, bn: int = 256) -> None:
+    """The rows of ``a`` (sorted by expert; ``moe_sort`` with tiles of ``gemm_tcgen05_tile_rows`` rows made ``tiles``), each by
+    the weights of its expert (``w`` [experts, N, K]), on the fifth-generation tensor cores.  Row pos goes to row
+    ``place``[pos] of ``c`` (None: pos).  ``epi``: "f32" store, "relu2", or "silu_mul" with the activation ``act``."""
+    experts, n, k = w.shape
+    rows = a.shape[0]
+    assert a.dtype is torch.bfloat16 and w.dtype is torch.bfloat16 and w.is_contiguous() and a.stride(1) == 1 and a.shape[1] == k
+    assert c.stride(1) == 1 and c.shape == (rows, n // 2 if epi == "silu_mul" else n)
+    assert c.dtype is (torch.float32 if epi == "f32" else torch.bfloat16) and epi in ("f32", "relu2", "silu_mul")
+    assert tiles.dtype is torch.int32 and tiles.is_contiguous() and tiles.shape[1] == 4
+    assert place is None or (place.dtype is torch.int32 and place.is_contiguous() and place.numel() >= rows)
+    _check(tcgen05_library().ie_gemm_tcgen05_grouped(_ptr(a), _ptr(w), _ptr(c), _ptr(tiles), _ptr(place), tiles.shape[0], rows,
+                                                     experts, n, k, a.stride(0), c.stride(0), _EPI[epi], bn, sm_count(),
+                                                     *_act4(act), _stream()),
+           f"gemm_tcgen05_grouped(rows={rows}, experts={experts}, n={n}, k={k}, {epi})")
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epi: str = "bf16", bn: int = 256,

@@ -11,8 +11,10 @@ Per token, with x the part's input (``RoutedExpertsSpec`` states the rule in ful
 
 The router's product also carries the shared expert's gate, if there is one (one more row).  Nothing waits for the device: the
 (token, choice) pairs are sorted by expert in one small kernel, and two grouped products walk the sorted pairs in
-tiles that never span two experts (``csrc/routed.cu``), so the part may sit inside a captured decode step.  A
-pair's result does not depend on where it lands in the sorted order, nor on what else the step holds.
+tiles that never span two experts (``csrc/routed.cu``), so the part may sit inside a captured decode step.  Prompt
+portions in bfloat16 that give the experts enough rows run both products on the tcgen05 tensor cores, over rows gathered
+into sorted order; a few tokens stream the chosen experts' weights.  A pair's result does not depend on where it lands in
+the sorted order, nor (beyond the rounding of another kernel's order of sums) on what else the step holds.
 """
 
 from __future__ import annotations
@@ -95,6 +97,14 @@ class RoutedExperts:
             self.correction = tensors[spec.router_bias].contiguous()      # the route kernel adds it to the logits
         self.shared = build_feedforward(spec.shared, tensors, rt) if spec.shared is not None else None
 
+    TCGEN05_MIN_ROWS = 32      # rows an expert gets on average from which tiles of 128 rows on tcgen05 pay
+
+    def _on_tcgen05(self, x: torch.Tensor, n_pairs: int) -> bool:
+        s = self.spec
+        return (self.rt.act_dtype is torch.bfloat16 and x.dtype is torch.bfloat16 and self.first.dtype is torch.bfloat16
+                and self.down.dtype is torch.bfloat16 and n_pairs >= self.TCGEN05_MIN_ROWS * s.n_experts and x.shape[0] >= 128
+                and s.hidden % 64 == 0 and s.intermediate % 64 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0)
+
     def _run_experts(self, x: torch.Tensor):
         """(the chosen experts' results [n * top, hidden] float32, their weights [n, top], the shared expert's gate)."""
         s, rt, ws = self.spec, self.rt, self.rt.ws
@@ -109,12 +119,21 @@ class RoutedExperts:
         kernels.moe_route(logits, self.correction, ids, weights, gate, E, top, s.n_groups, s.keep_groups, s.route_scale,
                           s.weight_eps, gate_col=E if self.gated_shared else -1, score=s.score, group_score=s.group_score)
         sorted_pairs = ws.take("moe_sorted", (n_pairs,), torch.int32)
+        hidden = ws.take("moe_hidden", (n_pairs, s.intermediate), rt.act_dtype)       # in sorted order
+        y = ws.take("moe_pairs_out", (n_pairs, s.hidden), torch.float32)               # in the pairs' own order
+        if self._on_tcgen05(x, n_pairs):
+            rows = kernels.gemm_tcgen05_tile_rows()
+            tiles = ws.take("moe_tiles", (kernels.moe_max_tiles(n_pairs, E, rows), 4), torch.int32)
+            kernels.moe_sort(ids, E, sorted_pairs, tiles, rows)
+            xs = ws.take("moe_rows", (n_pairs, s.hidden), torch.bfloat16)
+            kernels.moe_gather(x, xs, sorted_pairs, top)
+            kernels.gemm_tcgen05_grouped(xs, self.first, hidden, tiles, None, self.epi, act=self.act)
+            kernels.gemm_tcgen05_grouped(hidden, self.down, y, tiles, sorted_pairs, "f32")
+            return y, weights, gate
         tiles = ws.take("moe_tiles", (kernels.moe_max_tiles(n_pairs, E), 4), torch.int32)
         kernels.moe_sort(ids, E, sorted_pairs, tiles)
-        hidden = ws.take("moe_hidden", (n_pairs, s.intermediate), rt.act_dtype)       # in sorted order
         kernels.moe_gemm(x, self.first, hidden, sorted_pairs, tiles, top, gather=True, scatter=False, epi=self.epi,
                          act=self.act)
-        y = ws.take("moe_pairs_out", (n_pairs, s.hidden), torch.float32)               # in the pairs' own order
         kernels.moe_gemm(hidden, self.down, y, sorted_pairs, tiles, top, gather=False, scatter=True)
         return y, weights, gate
 

@@ -222,8 +222,9 @@ def test_activation_kernels_and_the_cap(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("d, ff, experts, top, shared", [(40, 24, 5, 2, 16), (72, 20, 3, 1, 0), (64, 136, 4, 3, 136), (64, 32, 6, 6, 200), (48, 40, 1, 1, 24)])
-@pytest.mark.parametrize("n", [1, 9, 150])
+@pytest.mark.parametrize("d, ff, experts, top, shared", [(40, 24, 5, 2, 16), (72, 20, 3, 1, 0), (64, 136, 4, 3, 136), (64, 32, 6, 6, 200),
+                                                         (48, 40, 1, 1, 24), (64, 128, 4, 3, 64), (192, 64, 7, 2, 128)])
+@pytest.mark.parametrize("n", [1, 9, 20, 150])
 def test_experts_without_a_gate_and_a_shared_one(dtype, d, ff, experts, top, shared, n):
     """Router, both grouped products on both of their kernels, the shared expert (a few rows and many), summed up by the
     part itself and left to the block."""
@@ -253,6 +254,109 @@ def test_experts_without_a_gate_and_a_shared_one(dtype, d, ff, experts, top, sha
     y, weights, more = part.forward_unsummed(x.to(DEV), None)
     total = (y.double().reshape(n, top, d) * weights.double()[:, :, None]).sum(1) + sum(m.double() for m in more)
     assert len(more) == bool(shared) and torch.allclose(total.cpu(), out, atol=1e-5, rtol=1e-5)
+
+
+@pytest.mark.parametrize("n, d, ff, experts, top", [(300, 128, 192, 5, 2), (700, 64, 64, 9, 3), (129, 320, 64, 3, 1), (260, 64, 320, 2, 2)])
+@pytest.mark.parametrize("bn", [128, 256])
+def test_grouped_product_on_tcgen05(n, d, ff, experts, top, bn):
+    """Experts with no row, with one, with exactly a tile's 128 and with several tiles; output widths that are no multiple
+    of a tile's; rows gathered into sorted order, results in sorted order and in the pairs' own places; every epilogue."""
+    bf = torch.bfloat16
+    g = torch.Generator().manual_seed(n + ff)
+    x = torch.randn(n, d, generator=g).to(bf)
+    first, both, down = ((torch.randn(experts, *s, generator=g) / s[-1] ** 0.5).to(bf) for s in ((ff, d), (2 * ff, d), (d, ff)))
+    ids = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(n)]).to(torch.int32)
+    if top == 1:
+        ids[:] = 2                                       # all in one expert, then one row and none in the others
+        ids[5] = 0
+    elif experts == 9:
+        ids[:, 0] = 8                                    # 700 rows of one expert; the others' counts follow from the rest
+        ids[:, 1] = torch.where(torch.arange(n) < 128, 1, 2)
+        ids[:, 2] = torch.where(torch.arange(n) < 1, 3, 4)
+    rows = k().gemm_tcgen05_tile_rows()
+    P = n * top
+    pairs = torch.empty(P, dtype=torch.int32, device=DEV)
+    tiles = torch.full((k().moe_max_tiles(P, experts, rows), 4), -5, dtype=torch.int32, device=DEV)
+    k().moe_sort(ids.to(DEV), experts, pairs, tiles, rows)
+    counts = torch.bincount(ids.flatten().long(), minlength=experts)
+    t, order = tiles.cpu(), pairs.cpu().long()
+    assert int(t[0, 3]) == int((t[:, 2] > 0).sum()) == int((-(-counts // rows)).sum()) and int(t[:, 2].sum()) == P
+    xs = torch.empty(P, d, dtype=bf, device=DEV)
+    k().moe_gather(x.to(DEV), xs, pairs, top)
+    assert torch.equal(xs.cpu(), x[order // top])
+    expert_of = ids.flatten().long()[order]
+    z = torch.einsum("pd,pfd->pf", xs.double().cpu(), first.double()[expert_of])
+    zb = torch.einsum("pd,pfd->pf", xs.double().cpu(), both.double()[expert_of])
+    h = torch.full((P, ff), float("nan"), dtype=bf, device=DEV)
+    k().gemm_tcgen05_grouped(xs, first.to(DEV), h, tiles, None, "relu2", bn=bn)
+    assert close(h, torch.relu(z) ** 2, "bfloat16", rel=1e-2)
+    for act in (None, k().glu_constants("gelu_tanh"), (1.702, 0.9, 1.0)):
+        k().gemm_tcgen05_grouped(xs, both.to(DEV), h, tiles, None, "silu_mul", act=act, bn=bn)
+        gate, up = zb[:, 0::2], zb[:, 1::2]
+        want = torch.nn.functional.silu(gate) * up if act is None else plain.gelu(gate) * up
+        if act is not None and len(act) == 3:
+            gate, up = gate.clamp(max=0.9), up.clamp(-0.9, 0.9)
+            want = gate * torch.sigmoid(1.702 * gate) * (up + 1)
+        assert close(h, want, "bfloat16", rel=1e-2), act
+    y = torch.full((P, d), float("nan"), device=DEV)
+    k().gemm_tcgen05_grouped(h, down.to(DEV), y, tiles, pairs, "f32", bn=bn)
+    torch.cuda.synchronize()
+    assert k().gemm_tcgen05_error() == 0
+    want = torch.empty(P, d, dtype=F)
+    want[order] = torch.einsum("pf,pdf->pd", h.double().cpu(), down.double()[expert_of])
+    assert torch.isfinite(y).all() and close(y, want, "bfloat16", rel=2e-3)
+    # the last rows of a wider result, and a result with a stride of its own
+    wide = torch.full((P, d + 8), 3.0, device=DEV)
+    k().gemm_tcgen05_grouped(h, down.to(DEV), wide[:, 4:4 + d], tiles, pairs, "f32", bn=bn)
+    assert torch.equal(wide[:, 4:4 + d], y) and bool((wide[:, :4] == 3.0).all()) and bool((wide[:, 4 + d:] == 3.0).all())
+
+
+@pytest.mark.parametrize("d, ff, experts, top, n", [(256, 64, 6, 2, 7), (72, 40, 4, 3, 16), (1024, 24, 3, 1, 1), (64, 520, 5, 5, 16)])
+def test_experts_products_that_stream_their_weights(d, ff, experts, top, n):
+    """The form for a few tokens beside the tiles' form, pair by pair, and against the plain products."""
+    bf = torch.bfloat16
+    g = torch.Generator().manual_seed(d + ff)
+    x = torch.randn(n, d, generator=g).to(bf)
+    first, down = ((torch.randn(experts, *s, generator=g) / s[-1] ** 0.5).to(bf) for s in ((2 * ff, d), (d, ff)))
+    ids = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(n)]).to(torch.int32)
+    pairs = torch.empty(n * top, dtype=torch.int32, device=DEV)
+    tiles = torch.empty(k().moe_max_tiles(n * top, experts), 4, dtype=torch.int32, device=DEV)
+    k().moe_sort(ids.to(DEV), experts, pairs, tiles)
+    order = pairs.cpu().long()
+    expert_of = ids.flatten().long()[order]
+    outs = []
+    for few in (True, False):
+        # the number of rows of the result decides: a result with rows to spare takes the other form
+        rows = n * top if few else (k().MOE_FEW_TOKENS + 1) * top
+        h, h2 = torch.zeros(rows, ff, dtype=bf, device=DEV), torch.zeros(rows, 2 * ff, dtype=bf, device=DEV)
+        y = torch.zeros(rows, d, device=DEV)
+        k().moe_gemm(x.to(DEV), first.to(DEV), h, pairs, tiles, top, gather=True, scatter=False, epi="silu_mul")
+        k().moe_gemm(x.to(DEV), first.to(DEV), h2, pairs, tiles, top, gather=True, scatter=False, epi="relu2")
+        k().moe_gemm(h, down.to(DEV), y, pairs, tiles, top, gather=False, scatter=True)
+        outs.append([t[:n * top].double().cpu() for t in (h, h2, y)])
+    z = torch.einsum("pd,pfd->pf", x.double()[order // top], first.double()[expert_of])
+    for h, h2, y in outs:
+        assert close(h, torch.nn.functional.silu(z[:, 0::2]) * z[:, 1::2], "bfloat16", rel=1e-2)
+        assert close(h2, torch.relu(z) ** 2, "bfloat16", rel=1e-2)
+        want = torch.empty(n * top, d, dtype=F)
+        want[order] = torch.einsum("pf,pdf->pd", h, down.double()[expert_of])
+        assert close(y, want, "bfloat16", rel=2e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("m, heads, kd, nd", [(1, 3, 10, 6), (8, 4, 192, 64), (16, 2, 64, 192), (9, 5, 17, 70), (3, 1, 300, 130), (12, 2, 40, 8)])
+def test_per_head_products_of_a_few_rows(dtype, m, heads, kd, nd):
+    dt = TORCH[dtype]
+    g = torch.Generator().manual_seed(kd)
+    x = torch.randn(m, heads * kd + 5, generator=g).to(dt)
+    w = (torch.randn(heads, kd, nd, generator=g) / kd ** 0.5).to(dt)
+    out = torch.full((m, heads * nd + 2), 7.0, dtype=dt, device=DEV)
+    k().heads_gemm(x.to(DEV)[:, :heads * kd], kd, w.to(DEV), out[:, :heads * nd], nd)
+    want = torch.einsum("mhk,hkn->mhn", x.double()[:, :heads * kd].reshape(m, heads, kd), w.double()).reshape(m, -1)
+    assert close(out[:, :heads * nd], want, dtype, rel=1e-2) and bool((out[:, heads * nd:] == 7.0).all())
+    alone = torch.empty(1, heads * nd, dtype=dt, device=DEV)      # a row's sum does not depend on the other rows
+    k().heads_gemm(x.to(DEV)[m - 1:, :heads * kd], kd, w.to(DEV), alone, nd)
+    assert torch.equal(alone[0], out[m - 1, :heads * nd])
 
 
 def test_router_of_sigmoid_scores_without_groups():
