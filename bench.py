@@ -1531,12 +1531,13 @@ def run_family(args):
                                                    k_gain=lg, k_norm_dims=kr, eps=1e-5, inv_freq=inv_l, rot_dims=r, q_rot_off=hd, k_rot_off=kr,
                                                    neighbours=True, mult=1.1)),
                 n * kr * 2 * 2, n * (H * (hd + r) * 2 + (kr + r) * 2) * 2)
-            kw = (lambda f, f2: dict(flops=n * f, flops_like=n * f2)) if n == N else (lambda f, f2: dict(nbytes=f, nbytes_like=f2))   # (bytes of the weights)
+            # these products are bound by the bytes of their operands: so few numbers a head are summed
+            nb = lambda k_, n_: H * (n * (k_ + n_) + k_ * n_) * 2
             add(f"queries into the compressed space, a product a head, {what}", "the same with a rotated part",
                 timed(lambda: heads_product(qp[:n], hd, absorb, qc[:n], kr)), timed(lambda: heads_product(ql[:n], hd + r, absorb2, qc2[:n], kr + r)),
-                **kw(2 * H * hd * kr, 2 * H * (hd + r) * (kr + r)))
+                nb(hd, kr), nb(hd + r, kr + r))
             add(f"values out of the compressed space, a product a head, {what}", "the same", *[timed(lambda: heads_product(mixed[:n], kr, expand, heads_out[:n], hd))] * 2,
-                **kw(2 * H * hd * kr, 2 * H * hd * kr))
+                nb(kr, hd))
             kw = dict(flops=4 * H * kr * pairs_all, flops_like=2 * H * (2 * kr + r) * pairs_all) if n == N else dict(nbytes=B * N * kr * 2, nbytes_like=B * N * (kr + r) * 2)
             add(f"latent attention, {what} ({H} heads over one row of {kr}, every key)", f"latent attention (rows of {kr + r})",
                 timed(lambda: lat(ctx, n), reps=5), timed(lambda: lat2(ctx, n), reps=5), **kw)
@@ -1563,18 +1564,36 @@ def run_family(args):
         route()
         up, gate_up, down = ((rnd(E, *s_) * 0.1).to(bf) for s_ in ((ffe, W), (2 * ffe, W), (W, ffe)))
         hid = torch.empty(N * top, ffe, device=dev, dtype=bf)
+        rows_tc = kernels.gemm_tcgen05_tile_rows()
+        xs = torch.empty(N * top, W, device=dev, dtype=bf)
         for n, _, what in both:
+            tile_rows = rows_tc if n == N else kernels.moe_tile_rows()
             pairs_ = torch.empty(n * top, dtype=torch.int32, device=dev)
-            tiles = torch.empty(kernels.moe_max_tiles(n * top, E), 4, dtype=torch.int32, device=dev)
-            kernels.moe_sort(ids[:n], E, pairs_, tiles)
+            tiles = torch.empty(kernels.moe_max_tiles(n * top, E, tile_rows), 4, dtype=torch.int32, device=dev)
+            kernels.moe_sort(ids[:n], E, pairs_, tiles, tile_rows)
             chosen = len(set(ids[:n].flatten().tolist()))
-            kw = (lambda k_: dict(flops=2 * n * top * ffe * W, flops_like=2 * n * top * k_ * ffe * W)) if n == N \
-                else (lambda k_: dict(nbytes=chosen * ffe * W * 2, nbytes_like=chosen * k_ * ffe * W * 2))
+            if n == N:
+                # prompt: rows gathered into sorted order, then the grouped product on tcgen05 | its tiles' form on mma.sync
+                tiles64 = torch.empty(kernels.moe_max_tiles(n * top, E), 4, dtype=torch.int32, device=dev)
+                add("rows gathered into sorted order, prompt", "a float32 scale in place", timed(lambda: kernels.moe_gather(x, xs, pairs_, top)),
+                    timed(lambda: kernels.scale_rows(pairs_y, 1.0)), n * W * 2 + n * top * W * 2, n * top * W * 8)
+                add("experts' first product with the square of relu, prompt", "experts' gate/up product with SiLU",
+                    timed(lambda: kernels.gemm_tcgen05_grouped(xs, up, hid, tiles, None, "relu2")),
+                    timed(lambda: kernels.gemm_tcgen05_grouped(xs, gate_up, hid, tiles, None, "silu_mul")),
+                    flops=2 * n * top * ffe * W, flops_like=2 * n * top * 2 * ffe * W)
+                pairs64 = torch.empty(n * top, dtype=torch.int32, device=dev)
+                kernels.moe_sort(ids, E, pairs64, tiles64)
+                add("experts' second product, prompt", "the same on mma.sync tiles of 64 rows",
+                    timed(lambda: kernels.gemm_tcgen05_grouped(hid, down, pairs_y, tiles, pairs_, "f32")),
+                    timed(lambda: kernels.moe_gemm(hid, down, pairs_y, pairs64, tiles64, top, gather=False, scatter=True)), flops=2 * n * top * ffe * W)
+                continue
             add(f"experts' first product with the square of relu, {what}", "experts' gate/up product with SiLU",
                 timed(lambda: kernels.moe_gemm(x[:n], up, hid[:n * top], pairs_, tiles, top, gather=True, scatter=False, epi="relu2")),
-                timed(lambda: kernels.moe_gemm(x[:n], gate_up, hid[:n * top], pairs_, tiles, top, gather=True, scatter=False, epi="silu_mul")), **kw(2))
+                timed(lambda: kernels.moe_gemm(x[:n], gate_up, hid[:n * top], pairs_, tiles, top, gather=True, scatter=False, epi="silu_mul")),
+                chosen * ffe * W * 2, chosen * 2 * ffe * W * 2)
             add(f"experts' second product, {what}", "the same",
-                *[timed(lambda: kernels.moe_gemm(hid[:n * top], down, pairs_y[:n * top], pairs_, tiles, top, gather=False, scatter=True))] * 2, **kw(1))
+                *[timed(lambda: kernels.moe_gemm(hid[:n * top], down, pairs_y[:n * top], pairs_, tiles, top, gather=False, scatter=True))] * 2,
+                chosen * ffe * W * 2)
         lgt, like_x = rnd(B, FAMILY_VOCAB), rnd(B, FAMILY_VOCAB)
         add("cap of the logits, decode b8", "a float32 scale in place", timed(lambda: kernels.softcap(lgt, 30.0)), timed(lambda: kernels.scale_rows(like_x, 1.0)),
             B * FAMILY_VOCAB * 8)
